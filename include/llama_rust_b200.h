@@ -100,7 +100,7 @@ int llr_exec_counters(const llr_exec* exec, llr_counters* out);
  * it cannot take), 3 = the integer tensor-core kernel for any number of
  * activation rows (f32-faithful), 4 = the tcgen05 GEMM whenever it can take
  * the call.  Automatic choice: up to 63 activation rows as 3, from 64 rows the
- * tcgen05 GEMM for every block-quantized format (16-bit operands, binary16 when
+ * tcgen05 GEMM for every block-quantized format and for BF16 (16-bit operands, binary16 when
  * the weights' range allows, else bfloat16: relative L2 error of a result up to
  * 4e-3 against the f32 row kernels, 3e-4 typical with binary16).
  * Also read once from the environment variable LLR_GEMV_PATH
@@ -547,6 +547,78 @@ int llr_session_seq_reset(llr_session* session, size_t seq);
  * the device half of prompt reuse [KvCache::prompt keeps the longest common prefix and recomputes the remainder,
  * langtax/tests/native_cuda_parity.rs:243-256]. */
 int llr_session_seq_truncate(llr_session* session, size_t seq, size_t n_keep);
+
+/* Logits at chosen rows of a ragged batch: as llr_session_batch, and for each of the n_want entries of `want` -- indices
+ * into `tokens`, in any order -- one row of n_vocab floats at `logits` (host), in the order of `want`.  n_want may be 0. */
+int llr_session_batch_rows(llr_session* session, size_t n_groups, const uint32_t* seq_ids, const uint32_t* counts,
+                           const int32_t* tokens, size_t n_want, const uint32_t* want, float* logits);
+/* Most rows one batch may have. */
+int llr_session_max_batch(const llr_session* session, size_t* rows);
+
+/* ---- decoders described layer by layer -------------------------------------------------------------------
+ * Sessions for decoder-only models outside the Llama walk: every layer names its mixer and its feed-forward, with their
+ * sizes and constants.  No counterpart in the reference, whose architectures are fixed walks.  Such a session has the
+ * same paged KV pool, batches, prompt reuse and greedy decode as a Llama session: all llr_session_* calls apply.  With
+ * llr_exec_set_path(exec, 3) everything is computed in f32; on the automatic path BF16 products of 16 rows and more run
+ * on the tensor cores with bfloat16 activations, and prompt chunks of 16 rows and more run their attention with binary16
+ * operands; norms, scores, softmax, gates and the residual stream are f32 either way.
+ *
+ * x = token_embd[token] * embd_scale (+ pos_embd[position]); per layer x += norm(mixer(x)), then x += norm(mlp(x)) when
+ * the layer has an mlp: the sublayers read x itself.  norm(y) = y / sqrt(mean(y^2) + norm_eps) * w, w as given here.
+ * logits = output (norm(x)).
+ *
+ * LLR_MIXER_ATTENTION: `in` stacks the rows q (n_head * dim) | k (n_head_kv * dim) | v (n_head_kv * vdim) | gate;
+ *   in_bias (NULL: none) holds the q | k | v rows' biases; q_norm / k_norm (NULL: none) weigh an RMS norm over ALL rows
+ *   of q / of k before they are split into heads.  score = (q . k) * scale + rel[bucket(distance)][head] when n_bucket > 0:
+ *   with h = n_bucket / 2, bucket(n) = n for n < h, else min(n_bucket - 1, h + floor(ln(n / h) / ln(bias_max / h) *
+ *   (n_bucket - h))).
+ * LLR_MIXER_LATENT: `in` stacks q (n_head * dim) | latent (kv_rank) | gate; the latent, RMS-normed with kv_norm, is what
+ *   the cache holds; keys are up_k latent, values up_v latent (BF16 matrices n_head * dim / n_head * vdim x kv_rank, head by head).
+ *   kv_from >= 0: no latent rows in `in`; the cached latents of that earlier latent layer are read instead.
+ * Both: window > 0: position i sees j with i - j < window, or j < keep_first; window 0: every earlier position.
+ *   LLR_GATE_ELEMENT (attention): the concatenated heads times sigmoid of n_head * vdim gate rows; LLR_GATE_HEAD (latent):
+ *   each head times sigmoid of its gate row.  `out`: n_embd x n_head * vdim.
+ * mlp: n_ff 0: none.  gate_up stacks gate | up (2 n_ff x n_embd); a = min(gate, limit), b = clamp(up, -limit, limit);
+ *   y = down (a * sigmoid(alpha * a) * (b + shift)). */
+#define LLR_MIXER_ATTENTION 0
+#define LLR_MIXER_LATENT 1
+#define LLR_GATE_NONE 0
+#define LLR_GATE_ELEMENT 1
+#define LLR_GATE_HEAD 2
+typedef struct llr_mixer {
+  uint32_t kind, n_head, n_head_kv, dim, vdim, kv_rank;
+  uint32_t window, keep_first;
+  int32_t kv_from;
+  uint32_t gate;
+  float scale;
+  uint32_t n_bucket, bias_max;
+  const llr_matrix *in, *up_k, *up_v, *out;
+  const float *in_bias, *q_norm, *k_norm, *kv_norm; /* host, copied */
+  const float* rel;                                 /* host, n_bucket x n_head, copied */
+} llr_mixer;
+typedef struct llr_mlp {
+  uint32_t n_ff;
+  float limit, alpha, shift;
+  const llr_matrix *gate_up, *down;
+} llr_mlp;
+typedef struct llr_decoder_layer {
+  llr_mixer mixer;
+  llr_mlp mlp;
+  const float *mixer_norm, *mlp_norm; /* host, n_embd floats, copied */
+} llr_decoder_layer;
+typedef struct llr_decoder_model {
+  uint32_t n_layer, n_embd, n_vocab, n_ctx;
+  float norm_eps, embd_scale;
+  const llr_matrix* token_embd; /* BF16 */
+  const llr_matrix* pos_embd;   /* BF16, at least n_ctx rows, or NULL */
+  const llr_matrix* output;     /* NULL: token_embd */
+  const float* output_norm;
+  const llr_decoder_layer* layers;
+} llr_decoder_model;
+int llr_session_create_decoder(llr_exec* exec, const llr_decoder_model* model, size_t n_seq, size_t kv_blocks,
+                               size_t block_tokens, llr_session** out);
+/* Copies the residual stream of the last batch's first n_rows rows (n_rows x n_embd floats) to the host. */
+int llr_session_residual(llr_session* session, size_t n_rows, float* out, size_t out_len);
 
 /* Dequantize rows [row0, row0+n_rows) of a resident matrix to f32 on the
  * device and copy them to out (n_rows*cols floats, host).  Bit-exact

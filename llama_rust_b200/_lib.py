@@ -28,7 +28,8 @@ SYMBOLS = [
     "llr_gguf_last_error", "llr_gguf_info", "llr_gguf_tensor_at", "llr_gguf_find", "llr_gguf_read", "llr_gguf_kv_u32",
     "llr_gguf_kv_f32", "llr_gguf_kv_bits", "llr_gguf_kv_bool", "llr_gguf_kv_string", "llr_gguf_kv_i32s", "llr_gguf_kv_type",
     "llr_gguf_upload", "llr_gguf_matmul", "llr_gguf_key", "llr_moe_ep_arena_bytes", "llr_moe_ep_create", "llr_moe_ep_dispatch",
-    "llr_moe_ep_serve", "llr_moe_ep_combine", "llr_moe_ep_run", "llr_moe_ep_free",
+    "llr_moe_ep_serve", "llr_moe_ep_combine", "llr_moe_ep_run", "llr_moe_ep_free", "llr_session_create_decoder",
+    "llr_session_batch_rows", "llr_session_max_batch", "llr_session_residual",
 ]
 ARENA_HEADER_BYTES = 65536
 
@@ -76,6 +77,28 @@ class LlamaLayer(C.Structure):
 class LlamaModel(C.Structure):
     _fields_ = [("cfg", LlamaConfig), ("token_embd", C.c_void_p), ("output", C.c_void_p), ("output_norm", C.c_void_p),
                 ("layers", C.POINTER(LlamaLayer))]
+
+
+class Mixer(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("kind", "n_head", "n_head_kv", "dim", "vdim", "kv_rank", "window", "keep_first")] + \
+               [("kv_from", C.c_int32), ("gate", C.c_uint32), ("scale", C.c_float), ("n_bucket", C.c_uint32), ("bias_max", C.c_uint32)] + \
+               [(n, C.c_void_p) for n in ("in_", "up_k", "up_v", "out", "in_bias", "q_norm", "k_norm", "kv_norm", "rel")]
+
+
+class Mlp(C.Structure):
+    _fields_ = [("n_ff", C.c_uint32), ("limit", C.c_float), ("alpha", C.c_float), ("shift", C.c_float),
+                ("gate_up", C.c_void_p), ("down", C.c_void_p)]
+
+
+class DecoderLayer(C.Structure):
+    _fields_ = [("mixer", Mixer), ("mlp", Mlp), ("mixer_norm", C.c_void_p), ("mlp_norm", C.c_void_p)]
+
+
+class DecoderModel(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("n_layer", "n_embd", "n_vocab", "n_ctx")] + \
+               [("norm_eps", C.c_float), ("embd_scale", C.c_float)] + \
+               [(n, C.c_void_p) for n in ("token_embd", "pos_embd", "output", "output_norm")] + \
+               [("layers", C.POINTER(DecoderLayer))]
 
 
 class MoeLayer(C.Structure):
@@ -164,6 +187,10 @@ def load() -> C.CDLL:
     lib.llr_session_create.argtypes = [vp, C.POINTER(LlamaModel), C.POINTER(vp)]
     lib.llr_session_create_paged.argtypes = [vp, C.POINTER(LlamaModel), sz, sz, sz, C.POINTER(vp)]
     lib.llr_session_batch.argtypes = [vp, sz, vp, vp, vp, vp, vp]
+    lib.llr_session_create_decoder.argtypes = [vp, C.POINTER(DecoderModel), sz, sz, sz, C.POINTER(vp)]
+    lib.llr_session_batch_rows.argtypes = [vp, sz, vp, vp, vp, sz, vp, vp]
+    lib.llr_session_max_batch.argtypes = [vp, C.POINTER(sz)]
+    lib.llr_session_residual.argtypes = [vp, sz, vp, sz]
     lib.llr_session_seq_position.argtypes = [vp, sz, C.POINTER(sz)]
     lib.llr_session_seq_reset.argtypes = [vp, sz]
     lib.llr_session_seq_truncate.argtypes = [vp, sz, sz]

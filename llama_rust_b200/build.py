@@ -51,11 +51,25 @@ def build(verbose: bool = False, ptxas_info: bool = False) -> str:
                 raise RuntimeError(f"nvcc failed on {src}")
     objs = [os.path.join(OBJ, os.path.basename(s)[:-3] + ".o") for s in sources]
     if _newer(objs, LIB):
-        cmd = [NVCC, "-shared", "-o", LIB, *objs, "-lcudart"]
+        part = LIB + ".part"  # a build that is interrupted leaves no half-written library behind
+        cmd = [NVCC, "-shared", "-o", part, *objs, "-lcudart"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
+        os.replace(part, LIB)
+    return LIB
+
+
+def ensure() -> str:
+    """The library, built first when the checkout has none (one process at a time builds)."""
+    if not os.path.exists(LIB):
+        import fcntl
+        os.makedirs(OBJ, exist_ok=True)
+        with open(os.path.join(OBJ, ".lock"), "w") as lock:
+            fcntl.flock(lock, fcntl.LOCK_EX)
+            if not os.path.exists(LIB):
+                build()
     return LIB
 
 

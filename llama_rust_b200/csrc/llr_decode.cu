@@ -11,51 +11,18 @@
 #include <cuda_runtime.h>
 
 #include <algorithm>
-#include <cstdlib>
 #include <math_constants.h>
 
+#include "llr_attend.cuh"
 #include "llr_kernels.cuh"
 
 namespace llr {
 namespace {
 
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(~0u, v, o);
-  return v;
-}
-__device__ __forceinline__ float warp_max(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(~0u, v, o));
-  return v;
-}
-// block-wide sum / max through shared memory (blockDim.x a multiple of 32, at most 1024); every thread gets the result
-__device__ __forceinline__ float block_sum(float v, float* sh) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  v = warp_sum(v);
-  __syncthreads();
-  if (lane == 0) sh[warp] = v;
-  __syncthreads();
-  float t = 0.f;
-  for (int w = 0; w < nw; ++w) t += sh[w];  // fixed order
-  return t;
-}
-
-__device__ __forceinline__ int row_position(const RowMap& r, int t) { return r.row_pos ? r.row_pos[t] : *r.pos_dev + t; }
-__device__ __forceinline__ int row_sequence(const RowMap& r, int t) { return r.row_seq ? r.row_seq[t] : 0; }
 // first float of the head vector of (sequence, layer, kv head, position) in a paged cache
 __device__ __forceinline__ int64_t kv_offset(const KvView& kv, int seq, int layer, int head, int pos, int n_head_kv, int hd) {
   const int b = kv.table[(int64_t)seq * kv.max_blocks + pos / kv.block_tokens];
   return ((((int64_t)b * kv.n_layer + layer) * n_head_kv + head) * kv.block_tokens + pos % kv.block_tokens) * hd;
-}
-
-// The element-wise kernels of the walk are launched with programmatic stream serialization: a kernel may be placed on
-// the SMs while its predecessor still runs, so its launch latency overlaps the predecessor's execution.  Each kernel
-// therefore waits for its predecessor (and everything before it) before it reads anything, and lets its successor be
-// placed right away; the matrix kernels that follow use that to prefetch weights.
-__device__ __forceinline__ void pdl_enter() {
-  asm volatile("griddepcontrol.wait;" ::: "memory");
-  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
 }
 
 // one block per activation row; a row of up to 4096 values stays in registers between the two passes
@@ -157,16 +124,16 @@ rope_store_kernel(float* __restrict__ q, float* __restrict__ k, const float* __r
 // `KV` says where the key and value rows of a position lie: in the paged cache (one row per block: decode steps) or
 // in a shared-memory tile that a block fills once for many rows of a prompt chunk.  The arithmetic is this one
 // function either way, so both kernels give the same bits.
-constexpr int ATT_THREADS = 256;
-constexpr int ATT_MAX_GQA = 8;
 constexpr int ATT_ROWS = 16;       // rows per block of the tiled kernel
 constexpr int ATT_TILE_CHUNK = 128; // longest slice the tiled kernel stages (2 x 128 x head_dim floats: contexts up to 4096 positions)
 
 struct KvGlobal {
   const KvView& kv;
   int sid, layer, hkv, n_head_kv, hd;
+  float scale;
   __device__ __forceinline__ const float* k(int s) const { return kv.k + kv_offset(kv, sid, layer, hkv, s, n_head_kv, hd); }
   __device__ __forceinline__ const float* v(int s) const { return kv.v + kv_offset(kv, sid, layer, hkv, s, n_head_kv, hd); }
+  __device__ __forceinline__ float score(int, int, float dot) const { return __fmul_rn(dot, scale); }
 };
 struct KvTile {
   const float* kt;
@@ -175,115 +142,6 @@ struct KvTile {
   __device__ __forceinline__ const float* k(int s) const { return kt + (s - s0) * hd; }
   __device__ __forceinline__ const float* v(int s) const { return vt + (s - s0) * hd; }
 };
-
-// sq: the row's query heads of this kv head [gqa][hd] in shared memory (filled and synchronized by the caller);
-// sc: [max(gqa * max_chunk, P * gqa * hd)] floats of shared memory; out: the slice's record of this row.
-// Ends with the block's threads past their last read of sq and sc only after the caller's next __syncthreads().
-template <typename KV>
-__device__ __forceinline__ void attend_slice(const KV& src, const float* sq, float* sc, float* out, int s0, int s1, int max_chunk,
-                                             int hd, int gqa) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = ATT_THREADS / 32;
-  const float scale = 1.0f / sqrtf((float)hd);
-  // scores: one warp per position, all query heads of the group against one read of the K row.  Four positions are in
-  // flight per warp (their K rows are fetched before any of them is used): the loop is bound by memory latency, not
-  // by arithmetic.  Each position's sum is formed exactly as if it were alone: columns in ascending order per lane.
-  constexpr int SP = 4;
-  for (int sbase = s0 + warp; sbase < s1; sbase += nw * SP) {
-    float acc[SP][ATT_MAX_GQA];
-    const float* krow[SP];
-#pragma unroll
-    for (int j = 0; j < SP; ++j) {
-      const int sj = sbase + j * nw;
-      krow[j] = sj < s1 ? src.k(sj) : nullptr;
-#pragma unroll
-      for (int g = 0; g < ATT_MAX_GQA; ++g) acc[j][g] = 0.f;
-    }
-    for (int i0 = 0; i0 < hd; i0 += 128) {
-      float kvv[SP][4];
-#pragma unroll
-      for (int j = 0; j < SP; ++j)
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int i = i0 + lane + 32 * u;
-          kvv[j][u] = (krow[j] && i < hd) ? krow[j][i] : 0.f;
-        }
-#pragma unroll
-      for (int j = 0; j < SP; ++j)
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          const int i = i0 + lane + 32 * u;
-          if (krow[j] && i < hd) {
-#pragma unroll
-            for (int g = 0; g < ATT_MAX_GQA; ++g)
-              if (g < gqa) acc[j][g] = fmaf(sq[g * hd + i], kvv[j][u], acc[j][g]);
-          }
-        }
-    }
-#pragma unroll
-    for (int j = 0; j < SP; ++j) {
-      const int sj = sbase + j * nw;
-      if (sj < s1) {  // warp-uniform
-#pragma unroll
-        for (int g = 0; g < ATT_MAX_GQA; ++g)
-          if (g < gqa) {
-            const float d = warp_sum(acc[j][g]);
-            if (lane == 0) sc[g * max_chunk + (sj - s0)] = __fmul_rn(d, scale);
-          }
-      }
-    }
-  }
-  __syncthreads();
-  // per query head: the slice's maximum and the sum of exp(score - max); one warp per head, lanes add in a fixed tree
-  for (int g = warp; g < gqa; g += nw) {
-    float m = -CUDART_INF_F;
-    for (int s = lane; s < s1 - s0; s += 32) m = fmaxf(m, sc[g * max_chunk + s]);
-    m = warp_max(m);
-    float l = 0.f;
-    for (int s = lane; s < s1 - s0; s += 32) {
-      const float e = expf(sc[g * max_chunk + s] - m);
-      sc[g * max_chunk + s] = e;
-      l += e;
-    }
-    l = warp_sum(l);
-    if (lane == 0) { out[g * (hd + 2) + hd] = m; out[g * (hd + 2) + hd + 1] = l; }
-  }
-  __syncthreads();
-  // weighted values: thread (i, grp) owns dimension i for every P-th run of eight positions of the slice
-  // (P = ATT_THREADS / hd thread groups); the groups' sums are added in group order through shared memory
-  const int P = ATT_THREADS / hd > 0 ? ATT_THREADS / hd : 1;
-  float acc[ATT_MAX_GQA];
-#pragma unroll
-  for (int g = 0; g < ATT_MAX_GQA; ++g) acc[g] = 0.f;
-  const int i = threadIdx.x % hd, grp = threadIdx.x / hd;
-  if (grp < P) {
-    // runs of eight positions go to the groups in turn: the split does not depend on the KV block size.  The eight
-    // value rows of a run are fetched before the first is used; the sums are formed in ascending position order.
-    for (int sb = s0 + 8 * grp; sb < s1; sb += 8 * P) {
-      float vv[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) vv[j] = sb + j < s1 ? src.v(sb + j)[i] : 0.f;
-#pragma unroll
-      for (int j = 0; j < 8; ++j)
-        if (sb + j < s1) {
-#pragma unroll
-          for (int g = 0; g < ATT_MAX_GQA; ++g)
-            if (g < gqa) acc[g] = fmaf(sc[g * max_chunk + (sb + j - s0)], vv[j], acc[g]);
-        }
-    }
-  }
-  __syncthreads();  // the scores are no longer needed: their space takes the groups' partial sums
-  float* vsum = sc;  // [P][gqa][hd]
-  if (grp < P)
-#pragma unroll
-    for (int g = 0; g < ATT_MAX_GQA; ++g)
-      if (g < gqa) vsum[(grp * gqa + g) * hd + i] = acc[g];
-  __syncthreads();
-  for (int idx = threadIdx.x; idx < gqa * hd; idx += ATT_THREADS) {
-    float v = 0.f;
-    for (int p = 0; p < P; ++p) v += vsum[p * gqa * hd + idx];
-    out[(idx / hd) * (hd + 2) + idx % hd] = v;
-  }
-}
 
 // The rotation of rope_store_kernel on n_vec vectors of hd floats in shared memory: one thread per pair
 __device__ __forceinline__ void rope_in_place(float* vecs, int n_vec, int hd, int pos, float theta_scale) {
@@ -338,7 +196,7 @@ attention_partial_kernel(const float* __restrict__ q, KvView kv, float* __restri
   }
   __syncthreads();
   float* out = part + (((int64_t)t * w.n_head_kv + hkv) * n_split + split) * gqa * (hd + 2);
-  attend_slice(KvGlobal{kv, sid, layer, hkv, w.n_head_kv, hd}, sq, sc, out, s0, s1, chunk, hd, gqa);
+  attend_slice<ATT_THREADS>(KvGlobal{kv, sid, layer, hkv, w.n_head_kv, hd, 1.0f / sqrtf((float)hd)}, sq, sc, out, s0, s1, chunk, hd, hd, gqa);
 }
 
 // The same slice of one row done by ONE warp, every elementary sum formed in the order attend_slice forms it (a
@@ -860,26 +718,6 @@ int attention_chunk(const WalkShape& w) {
 int attention_splits(const WalkShape& w) {
   const int c = attention_chunk(w);
   return (w.n_ctx + c - 1) / c;
-}
-
-// LLR_WALK_PDL=0 launches these kernels in plain stream order
-bool walk_pdl() {
-  static const bool on = [] { const char* v = std::getenv("LLR_WALK_PDL"); return !(v && v[0] == '0'); }();
-  return on;
-}
-template <typename... P, typename... A>
-cudaError_t launch_walk(void (*kern)(P...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, A... args) {
-  cudaLaunchAttribute attr;
-  attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr.val.programmaticStreamSerializationAllowed = 1;
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = grid;
-  cfg.blockDim = block;
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = s;
-  cfg.attrs = &attr;
-  cfg.numAttrs = walk_pdl() ? 1 : 0;
-  return cudaLaunchKernelEx(&cfg, kern, static_cast<P>(args)...);
 }
 
 }  // namespace

@@ -302,7 +302,7 @@ cudaError_t ensure_scratch(llr_exec* e, const llr_matrix* m, size_t tokens, void
   *out = nullptr;
   const MatView v = view_of(m);
   if (!matmul_wants_tc(v, (int64_t)tokens, e->path)) return cudaSuccess;
-  cudaError_t ce = grow_device(&e->dev_s, &e->dev_s_cap, gemm_tc_scratch_bytes(v, (int64_t)tokens));
+  cudaError_t ce = grow_device(&e->dev_s, &e->dev_s_cap, matmul_scratch_bytes(v, (int64_t)tokens));
   if (ce == cudaSuccess) *out = e->dev_s;
   return ce;
 }
@@ -429,16 +429,30 @@ int run_host(llr_exec* e, const llr_matrix* m, size_t tokens, const float* x, fl
 
 namespace llr {
 
+static bool bf16_chunk(const MatView& m, int64_t tokens) {
+  return m.dtype == LLR_DTYPE_BF16 && tokens >= BF16_TC_MIN_TOKENS && tokens <= (1 << 24) && gemm_bf16_supported(m.w, m.rows, m.cols);
+}
 bool matmul_wants_tc(const MatView& m, int64_t tokens, int path) {
-  if (path == PATH_TC) return gemm_tc_supported(m, tokens);
-  return path == PATH_AUTO && tokens >= TC_MIN_TOKENS && gemm_tc_supported(m, tokens);
+  if (path != PATH_TC && !(path == PATH_AUTO && tokens >= TC_MIN_TOKENS)) return false;
+  return gemm_tc_supported(m, tokens) || bf16_chunk(m, tokens);
+}
+size_t matmul_scratch_bytes(const MatView& m, int64_t tokens) {
+  return bf16_chunk(m, tokens) ? ((size_t)tokens * m.cols * 2 + 255) / 256 * 256 : gemm_tc_scratch_bytes(m, tokens);
 }
 
 cudaError_t launch_matmul(const MatView& m, const float* x, float* y, int64_t tokens,
                           cudaStream_t stream, int path, int sm_count, int* err_flag,
                           void* scratch, uint64_t* launches) {
   const bool x_aligned = ((uintptr_t)x & 15) == 0 && (m.cols % 4 == 0);
-  if (scratch && err_flag && x_aligned && matmul_wants_tc(m, tokens, path))
+  if (scratch && err_flag && x_aligned && ((uintptr_t)y & 15) == 0 && matmul_wants_tc(m, tokens, path) && bf16_chunk(m, tokens)) {
+    const cudaError_t ce = tc_convert_activations(x, tokens, (int)m.cols, false, scratch, nullptr, stream, launches);
+    if (ce != cudaSuccess) return ce;
+    Bf16Product p{};
+    p.w = m.w; p.x16 = scratch; p.x_ld = p.x_cols = m.cols; p.y = y; p.y_ld = m.rows;
+    p.tokens = (int)tokens; p.rows = (int)m.rows; p.cols = (int)m.cols; p.batch = 1; p.slices = 1;
+    return launch_gemm_bf16(p, stream, err_flag, launches);
+  }
+  if (scratch && err_flag && x_aligned && matmul_wants_tc(m, tokens, path) && gemm_tc_supported(m, tokens))
     return launch_gemm_tc(m, x, y, tokens, scratch, gemm_tc_scratch_bytes(m, tokens), stream, err_flag, launches);
   if (path == PATH_TC) path = PATH_AUTO;
   if ((path == PATH_AUTO || path == PATH_MMA) && x_aligned && err_flag && gemv_mma_supported(m))
@@ -1580,6 +1594,8 @@ int llr_program_free(llr_program* p) {
 }
 
 // ---------------------------------------------------------------- device-resident Llama walk
+namespace { struct LayeredDecoder; }
+
 struct llr_session {
   llr_exec* owner = nullptr;
   llr_llama_config cfg{};
@@ -1619,6 +1635,7 @@ struct llr_session {
   };
   std::vector<std::unique_ptr<Moe>> moe;  // per layer, null: dense FFN
   std::vector<std::pair<size_t, size_t>> batch_groups;  // llr_session_batch: (first row, rows) of each group of the batch in flight
+  std::unique_ptr<LayeredDecoder> dec;  // a decoder described layer by layer (null: the Llama walk)
   bool has_moe = false, moe_select = false;  // moe_select: every routed layer can choose its experts' products on the device
   int* moe_sel = nullptr;     // one token's experts in ascending id (8 ints), then their router weights (8 floats)
   float* moe_y = nullptr;     // the selected experts' down results (8 x n_embd)
@@ -1682,6 +1699,24 @@ int session_reserve(llr_session* s, size_t seq, size_t upto) {
   return LLR_OK;
 }
 
+// Sequences and their paged pool: n_seq sequences of at most n_ctx positions over kv_blocks blocks (0: enough for all).
+void session_pool(llr_session* s, size_t n_seq, size_t kv_blocks, size_t block_tokens) {
+  const size_t n_ctx = s->cfg.n_ctx;
+  s->max_batch = n_ctx * n_seq < 512 ? n_ctx * n_seq : 512;
+  s->n_seq = n_seq;
+  s->block_tokens = block_tokens;
+  s->max_blocks = (n_ctx + block_tokens - 1) / block_tokens;
+  s->n_blocks = kv_blocks ? kv_blocks : s->max_blocks * n_seq;
+  s->position.assign(n_seq, 0);
+  s->seq_blocks.assign(n_seq, {});
+  s->have_logits.assign(n_seq, 0);
+  for (size_t b = s->n_blocks; b-- > 0;) s->free_blocks.push_back((int)b);
+  s->logits_rows = n_seq;
+  if (const char* g = std::getenv("LLR_SESSION_GRAPH")) s->use_graph = s->use_graph && std::strcmp(g, "0") != 0;
+}
+
+#include "llr_layered.cuh"
+
 // The routed-expert layer of layer li over the n normalised rows in s->xn; the result (not yet added to the residual
 // stream) goes to s->proj.  The per-expert row counts visit the host, which sizes the expert launches with them.
 cudaError_t session_moe_ffn(llr_session* s, size_t li, size_t n) {
@@ -1743,6 +1778,10 @@ cudaError_t session_moe_ffn(llr_session* s, size_t li, size_t n) {
 // s->x and the last ffn_down result, not yet added, in s->proj (returned through *pending).
 cudaError_t session_layers(llr_session* s, const int* ids_dev, size_t n, const RowMap& rows, const float** pending_out) {
   llr_exec* e = s->owner;
+  if (s->dec) {
+    *pending_out = nullptr;
+    return layered_layers(s, ids_dev, n, rows);
+  }
   const llr_llama_config& c = s->cfg;
   const size_t E = c.n_embd, FF = c.n_ff;
   cudaStream_t st = e->stream;
@@ -1909,16 +1948,7 @@ int session_create(llr_exec* e, const llr_llama_model* m, size_t n_seq, size_t k
   const float n_rot = (float)(uint16_t)c.head_dim;
   s->shape = WalkShape{(int)c.n_embd, (int)c.n_head, (int)c.n_head_kv, (int)c.head_dim, (int)c.n_ff, (int)c.n_ctx, c.rms_eps, c.rope_base,
                        std::pow(c.rope_base, -2.0f / n_rot)};  // decode.rs:11578: theta_scale in f32
-  s->max_batch = c.n_ctx * n_seq < 512 ? c.n_ctx * n_seq : 512;
-  s->n_seq = n_seq;
-  s->block_tokens = block_tokens;
-  s->max_blocks = (c.n_ctx + block_tokens - 1) / block_tokens;
-  s->n_blocks = kv_blocks ? kv_blocks : s->max_blocks * n_seq;
-  s->position.assign(n_seq, 0);
-  s->seq_blocks.assign(n_seq, {});
-  s->have_logits.assign(n_seq, 0);
-  for (size_t b = s->n_blocks; b-- > 0;) s->free_blocks.push_back((int)b);
-  s->logits_rows = n_seq;
+  session_pool(s, n_seq, kv_blocks, block_tokens);
   const size_t B = s->max_batch;
   cudaError_t ce = cudaSuccess;
   auto alloc = [&](float** p, size_t n) { if (ce == cudaSuccess) ce = cudaMalloc((void**)p, n * sizeof(float)); };
@@ -1935,15 +1965,14 @@ int session_create(llr_exec* e, const llr_llama_model* m, size_t n_seq, size_t k
   norm(m->output_norm, &s->out_norm);
   alloc(&s->x, B * E); alloc(&s->xn, B * E); alloc(&s->q, B * QW); alloc(&s->k, B * KVW); alloc(&s->v, B * KVW);
   alloc(&s->attn, B * QW); alloc(&s->proj, B * E); alloc(&s->gate, B * FF); alloc(&s->up, B * FF);
-  alloc(&s->logits, s->logits_rows * V); alloc(&s->last_x, n_seq * E); alloc(&s->arg_part, 512);
+  alloc(&s->logits, s->logits_rows * V); alloc(&s->last_x, s->logits_rows * E); alloc(&s->arg_part, 512);
   const size_t pool = s->n_blocks * c.n_layer * c.n_head_kv * block_tokens * c.head_dim;
   alloc(&s->cache_k, pool); alloc(&s->cache_v, pool);
   alloc(&s->att_scratch, attention_scratch_floats((int)B, s->shape));
   ialloc(&s->pos_dev, 1); ialloc(&s->count_dev, 1);
-  ialloc(&s->table_dev, n_seq * s->max_blocks); ialloc(&s->row_pos, B); ialloc(&s->row_seq, B); ialloc(&s->last_rows, n_seq);
+  ialloc(&s->table_dev, n_seq * s->max_blocks); ialloc(&s->row_pos, B); ialloc(&s->row_seq, B); ialloc(&s->last_rows, s->logits_rows);
   if (ce == cudaSuccess) ce = cudaMemset(s->pos_dev, 0, sizeof(int));
   if (ce == cudaSuccess) ce = cudaMemset(s->table_dev, 0, n_seq * s->max_blocks * sizeof(int));
-  if (const char* g = std::getenv("LLR_SESSION_GRAPH")) s->use_graph = s->use_graph && std::strcmp(g, "0") != 0;
   if (max_expert > 0 && ce == cudaSuccess) {
     // One-token steps choose their experts' products on the device when every expert matrix of every routed layer goes
     // through the streaming decode kernel in one format per kind: tensor maps gate | up | down of all experts per layer.
@@ -2060,6 +2089,11 @@ int llr_session_create(llr_exec* e, const llr_llama_model* m, llr_session** out)
 int llr_session_create_paged(llr_exec* e, const llr_llama_model* m, size_t n_seq, size_t kv_blocks, size_t block_tokens,
                              llr_session** out) {
   return session_create(e, m, n_seq, kv_blocks, block_tokens, out);
+}
+
+int llr_session_create_decoder(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t kv_blocks, size_t block_tokens,
+                               llr_session** out) {
+  return layered_create(e, m, n_seq, kv_blocks, block_tokens, out);
 }
 
 int llr_session_free(llr_session* s) {
@@ -2237,8 +2271,10 @@ int llr_session_logits(llr_session* s, float* logits, size_t n) {
 // (Engine::try_compute_batch, engine.rs:1215-1274 -> prefill_batch decode.rs:2579); attention and the KV cache go by
 // each row's own sequence and position.  last_logits (optional, n_groups x n_vocab, in the caller's group order) and
 // next_ids (optional, n_groups) receive each group's last-row logits and their greedy argmax.
-int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, const uint32_t* counts, const int32_t* tokens,
-                      float* last_logits, int32_t* next_ids) {
+// Or, with `rows`: logits of the rows `want` names (indices into `tokens`).
+struct WantedRows { size_t n; const uint32_t* want; float* logits; };
+static int session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, const uint32_t* counts, const int32_t* tokens,
+                         const WantedRows* rows, float* last_logits, int32_t* next_ids) {
   if (!s || !s->owner) return LLR_ERR_INVALID;
   llr_exec* e = s->owner;
   if (n_groups == 0 || n_groups > s->n_seq || !seq_ids || !counts || !tokens) return fail(e, LLR_ERR_INVALID, "a batch needs 1..n_seq groups");
@@ -2258,6 +2294,11 @@ int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, 
   if (total > s->max_batch) return fail(e, LLR_ERR_INVALID, "the batch has more rows than the session's chunk size (" + std::to_string(s->max_batch) + ")");
   for (size_t i = 0; i < total; ++i)
     if (tokens[i] < 0 || (uint32_t)tokens[i] >= c.n_vocab) return fail(e, LLR_ERR_INVALID, "token id out of range");
+  if (rows && rows->n > 0) {
+    if (!rows->want || !rows->logits) return fail(e, LLR_ERR_INVALID, "wanted rows need an index list and a buffer");
+    for (size_t i = 0; i < rows->n; ++i)
+      if (rows->want[i] >= total) return fail(e, LLR_ERR_INVALID, "a wanted row lies outside the batch");
+  }
   DeviceGuard guard(e->device);
   int rc = session_ids(s, total);
   if (rc) return rc;
@@ -2265,7 +2306,7 @@ int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, 
   std::vector<size_t> order(n_groups);
   for (size_t g = 0; g < n_groups; ++g) order[g] = g;
   std::sort(order.begin(), order.end(), [&](size_t a, size_t b) { return seq_ids[a] < seq_ids[b]; });
-  std::vector<int> ids(total), rpos(total), rseq(total), last(n_groups);
+  std::vector<int> ids(total), rpos(total), rseq(total), last(n_groups), row_of(rows ? total : 0);
   size_t r = 0;
   s->batch_groups.clear();
   for (size_t oi = 0; oi < n_groups; ++oi) {
@@ -2274,6 +2315,7 @@ int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, 
     s->batch_groups.emplace_back(r, (size_t)counts[g]);
     for (size_t i = 0; i < counts[g]; ++i, ++r) {
       ids[r] = tokens[first[g] + i];
+      if (rows) row_of[first[g] + i] = (int)r;
       rpos[r] = (int)(s->position[q] + i);
       rseq[r] = (int)q;
     }
@@ -2292,7 +2334,21 @@ int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, 
     return fail_cuda(e, ce, "kernel launch");
   // each group's last row: residual add, output norm, logits (LogitsKind::Last per sequence)
   if (pending && (ce = launch_add(s->x, pending, (int64_t)(total * E), st, L)) != cudaSuccess) return fail_cuda(e, ce, "kernel launch");
-  if ((ce = launch_gather_rows(s->x, s->last_rows, s->last_x, (int)n_groups, (int)E, st, L)) != cudaSuccess ||
+  if (rows) {
+    std::vector<int> pick;
+    for (size_t w0 = 0; w0 < rows->n; w0 += s->logits_rows) {
+      const size_t nw = std::min(s->logits_rows, rows->n - w0);
+      pick.resize(nw);
+      for (size_t i = 0; i < nw; ++i) pick[i] = row_of[rows->want[w0 + i]];
+      if ((ce = cudaMemcpyAsync(s->last_rows, pick.data(), nw * sizeof(int), cudaMemcpyHostToDevice, st)) != cudaSuccess ||
+          (ce = launch_gather_rows(s->x, s->last_rows, s->last_x, (int)nw, (int)E, st, L)) != cudaSuccess ||
+          (ce = launch_rmsnorm(s->last_x, nullptr, s->out_norm, s->last_x, (int)nw, (int)E, c.rms_eps, st, L)) != cudaSuccess ||
+          (ce = session_matmul(e, s->output, nw, s->last_x, s->logits)) != cudaSuccess ||
+          (ce = cudaMemcpyAsync(rows->logits + w0 * V, s->logits, nw * V * sizeof(float), cudaMemcpyDeviceToHost, st)) != cudaSuccess ||
+          (ce = cudaStreamSynchronize(st)) != cudaSuccess)
+        return fail_cuda(e, ce, "logits of the wanted rows");
+    }
+  } else if ((ce = launch_gather_rows(s->x, s->last_rows, s->last_x, (int)n_groups, (int)E, st, L)) != cudaSuccess ||
       (ce = launch_rmsnorm(s->last_x, nullptr, s->out_norm, s->last_x, (int)n_groups, (int)E, c.rms_eps, st, L)) != cudaSuccess ||
       (ce = session_matmul(e, s->output, n_groups, s->last_x, s->logits)) != cudaSuccess)
     return fail_cuda(e, ce, "kernel launch");
@@ -2321,6 +2377,34 @@ int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, 
         (ce = cudaStreamSynchronize(st)) != cudaSuccess)
       return fail_cuda(e, ce, "position upload");
   }
+  return LLR_OK;
+}
+
+int llr_session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_ids, const uint32_t* counts, const int32_t* tokens,
+                      float* last_logits, int32_t* next_ids) {
+  return session_batch(s, n_groups, seq_ids, counts, tokens, nullptr, last_logits, next_ids);
+}
+
+int llr_session_batch_rows(llr_session* s, size_t n_groups, const uint32_t* seq_ids, const uint32_t* counts, const int32_t* tokens, size_t n_want,
+                           const uint32_t* want, float* logits) {
+  const WantedRows rows{n_want, want, logits};
+  return session_batch(s, n_groups, seq_ids, counts, tokens, &rows, nullptr, nullptr);
+}
+
+int llr_session_max_batch(const llr_session* s, size_t* rows) {
+  if (!s || !rows) return LLR_ERR_INVALID;
+  *rows = s->max_batch;
+  return LLR_OK;
+}
+
+int llr_session_residual(llr_session* s, size_t n_rows, float* out, size_t out_len) {
+  if (!s || !s->owner) return LLR_ERR_INVALID;
+  llr_exec* e = s->owner;
+  if (!out || n_rows > s->max_batch || out_len != n_rows * s->cfg.n_embd) return fail(e, LLR_ERR_INVALID, "residual buffer does not match the rows asked for");
+  DeviceGuard guard(e->device);
+  cudaError_t ce = cudaMemcpyAsync(out, s->x, out_len * sizeof(float), cudaMemcpyDeviceToHost, e->stream);
+  if (ce == cudaSuccess) ce = cudaStreamSynchronize(e->stream);
+  if (ce != cudaSuccess) return fail_cuda(e, ce, "residual download");
   return LLR_OK;
 }
 

@@ -45,11 +45,12 @@ constexpr int64_t TC_MIN_TOKENS = 64;  // from here on AUTO prefers the bf16 tcg
 // y[t*rows + r] = sum_c W[r,c] * x[t*cols + c] for t < tokens.  Any shape the
 // entry points accept.  `launches` is incremented by the kernels launched.
 // `err_flag` is a device int that kernels with bounded waits set to non-zero when a wait ran out.
-// `scratch` (gemm_tc_scratch_bytes, or null) lets the tensor-core GEMM stage bf16 activations.
+// `scratch` (matmul_scratch_bytes, or null) lets the tensor-core GEMM stage 16-bit activations.
 cudaError_t launch_matmul(const MatView& m, const float* x, float* y, int64_t tokens,
                           cudaStream_t stream, int path, int sm_count, int* err_flag,
                           void* scratch, uint64_t* launches);
 bool matmul_wants_tc(const MatView& m, int64_t tokens, int path);
+size_t matmul_scratch_bytes(const MatView& m, int64_t tokens);  // for launch_matmul when matmul_wants_tc
 
 // Always-available reference kernel: one warp per row, byte loads, any alignment.
 cudaError_t launch_gemv_generic(const MatView& m, const float* x, float* y, int64_t tokens,
@@ -298,6 +299,82 @@ cudaError_t launch_argmax_advance(const float* logits, int n, int* out_id, float
 // one argmax per row of logits[n_rows][n] -> out_id[row], out_margin[row] (optional)
 cudaError_t launch_argmax_rows(const float* logits, int n_rows, int n, int* out_id, float* out_margin, cudaStream_t s,
                                uint64_t* launches);
+
+// ---- products with bfloat16 weights for many rows (llr_gemm_bf16.cu): tcgen05, bfloat16 activations, f32 accumulation ----
+// y[t * y_ld + z * rows + r] = sum_c W[z * rows + r][c] x[t][z * xk + c] for z < batch (a product per head), times
+// sigmoid(gate[t * gate_ld + z]) when gate is set.  Results as f32 (y), as bfloat16 (y16), or both.  With slices > 1
+// (batch 1, y only) slice s of the K range leaves its partial sums at y + s * slice_stride.
+struct Bf16Product {
+  const void* w;      // [batch * rows][cols]
+  const void* x16;    // [tokens][x_ld], of which x_cols columns exist
+  int64_t x_ld, x_cols;
+  float* y;
+  void* y16;
+  const float* gate;
+  int64_t y_ld, gate_ld, slice_stride;
+  int tokens, rows, cols, batch, xk, slices;
+};
+bool gemm_bf16_supported(const void* w, int64_t rows, int64_t cols);
+int gemm_bf16_slices(int tokens, int rows, int cols);
+cudaError_t launch_gemm_bf16(const Bf16Product& p, cudaStream_t stream, int* err, uint64_t* launches);
+constexpr int BF16_TC_MIN_TOKENS = 16;  // from here on the walk of a layered decoder prefers it
+
+// ---- kernels of decoders described layer by layer (llr_mixers.cu) ----
+// A layer's keys and values in the paged pool: head vector of (block b, kv head g, position t of the block) lies at
+// k + b * k_block + (g * block_tokens + t) * dk, values likewise; a latent layer has one vector per position that serves
+// as key and value of every head (v == k).
+struct LayerKv {
+  float* k;
+  float* v;
+  const int* table;
+  int block_tokens, max_blocks;
+  int64_t k_block, v_block;
+};
+// What a row attends to and how it scores: n_head query heads over n_kv key/value heads (n_head / n_kv share one), the
+// last `window` positions (0: all) and the first keep_first; score = (q . k) * scale + bias[h][min(distance, bias_len - 1)].
+struct SpanShape {
+  int n_head, n_kv, dk, dv, window, keep_first, n_ctx;
+  float scale;
+  const float* bias;  // [n_head][bias_len], or null
+  int bias_len;
+};
+// x[t] = table[ids[t]] * scale + pos_table[position of t]; table and pos_table (may be null) are bfloat16 rows of n.
+// x16 (may be null): the same as bfloat16.
+cudaError_t launch_embed(const void* table, const void* pos_table, const int* ids, const RowMap& rows, float scale, float* x,
+                         void* x16, int tokens, int n, cudaStream_t s, uint64_t* launches);
+// q | k | v of a stacked projection (row t at proj + t * ld): bias added; q and k divided by the root mean square of the
+// WHOLE projection and weighted, where norms are given; k and v into the cache, q left in place.
+struct QkvShape { int n_head, n_kv, dk, dv; float eps; };
+cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh,
+                             const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
+// One latent per row (n floats at proj + t * ld): normed, weighted, into the cache.  q16 (may be null): the nq floats at
+// q + t * ld as bfloat16 rows of nq.
+cudaError_t launch_latent_store(const float* proj, int ld, const float* w, int n, float eps, const LayerKv& kv, const RowMap& rows,
+                                int tokens, cudaStream_t s, uint64_t* launches);
+cudaError_t launch_rows_bf16(const float* x, int64_t ld, int n, void* out16, int tokens, cudaStream_t s, uint64_t* launches);
+// Products per head with bfloat16 weights and f32 activations.
+// transposed: y[t][h * cols + c] = sum_r W[h * rows + r][c] x[t * x_ld + h * rows + r]     (a query into the latent space)
+// plain:      y[t][h * rows + r] = sum_c W[h * rows + r][c] x[t * x_ld + h * cols + c]     (a latent out of it), times
+//             sigmoid(gate[t * gate_ld + h]) when gate is set
+cudaError_t launch_head_product_t(const void* w, int heads, int rows, int cols, const float* x, int64_t x_ld, float* y, int tokens,
+                                  cudaStream_t s, uint64_t* launches);
+cudaError_t launch_head_product(const void* w, int heads, int rows, int cols, const float* x, int64_t x_ld, float* y, const float* gate,
+                                int64_t gate_ld, int tokens, cudaStream_t s, uint64_t* launches);
+cudaError_t launch_head_transpose(const void* w, int heads, int rows, int cols, void* out, cudaStream_t s, uint64_t* launches);
+// Attention over the visible keys.  q: row t at q + t * q_ld.  Result rows of n_head * dv, f32 (out) and/or bfloat16 (out16);
+// gate (may be null): element gate, result times sigmoid(gate[t * gate_ld + h * dv + i]).
+// one_sequence: the rows are one sequence at consecutive positions; with tensor_cores such rows may run as binary16 MMAs.
+size_t span_scratch_floats(const SpanShape& sh);
+bool span_supported(const SpanShape& sh);
+cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape& sh, const LayerKv& kv, const RowMap& rows, int t0, int tokens,
+                                  float* out, void* out16, const float* gate, int64_t gate_ld, float* scratch, bool tensor_cores,
+                                  bool one_sequence, cudaStream_t s, uint64_t* launches);
+// x[t] += y[t] / rms(y[t]) * w, y given as `slices` partial sums `slice_stride` floats apart; x16 (may be null): the new x
+cudaError_t launch_norm_add(float* x, const float* y, int slices, int64_t slice_stride, const float* w, float eps, void* x16, int tokens, int n,
+                            cudaStream_t s, uint64_t* launches);
+// out[t][i] = a * sigmoid(alpha * a) * (b + shift), a = min(gu[t][i], limit), b = clamp(gu[t][n + i], -limit, limit)
+struct GluShape { int n; float limit, alpha, shift; };
+cudaError_t launch_clamped_glu(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches);
 
 // *flag_dev = 1 when the two device byte ranges differ (both 16-byte aligned), else 0
 cudaError_t launch_bytes_differ(const void* a, const void* b, size_t n, int* flag_dev, cudaStream_t stream, uint64_t* launches);

@@ -1,0 +1,800 @@
+// Kernels of decoders described layer by layer: what stands between the matrix products of a layer whose mixer is
+// (a) attention over key/value heads with norms over the whole query / key projection, projection biases, a learned bias
+// per head and distance bucket, a sliding window that keeps the first tokens, and an element-wise output gate, or
+// (b) latent attention: one normed latent vector per position is cached and serves every head; a head's query is taken
+// into the latent space (q' = W_uk^T q, so that q . (W_uk c) = q' . c) and its result out of it (W_uv (sum p c)).
+// Then the norm on a sublayer's output with its residual add, the clamped gated unit, and the embedding with learned
+// positions.  Sizes and constants are arguments; a mechanism that is absent is a null pointer or a zero.
+//
+// Scores, softmax, norms, sigmoids and the residual stream are f32 throughout.
+#include <cuda_bf16.h>
+#include <cuda_fp16.h>
+#include <cuda_runtime.h>
+#include <math_constants.h>
+
+#include <algorithm>
+
+#include "llr_attend.cuh"
+#include "llr_kernels.cuh"
+
+namespace llr {
+namespace {
+
+__device__ __forceinline__ float bf(uint16_t v) { return __uint_as_float((uint32_t)v << 16); }
+__device__ __forceinline__ float sigmoid(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
+__device__ __forceinline__ uint2 pack4_bf16(float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  return make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
+}
+
+// ---- embedding ------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+embed_kernel(const uint16_t* __restrict__ table, const uint16_t* __restrict__ pos_table, const int* __restrict__ ids, RowMap rows, float scale,
+             float* __restrict__ x, __nv_bfloat16* __restrict__ x16, int n) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  const uint16_t* e = table + (int64_t)ids[t] * n;
+  const uint16_t* p = pos_table ? pos_table + (int64_t)row_position(rows, t) * n : nullptr;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    float v = __fmul_rn(bf(e[i]), scale);
+    if (p) v = __fadd_rn(v, bf(p[i]));
+    x[(int64_t)t * n + i] = v;
+    if (x16) x16[(int64_t)t * n + i] = __float2bfloat16_rn(v);
+  }
+}
+
+// ---- projections into the cache ---------------------------------------------------------------------------------
+__device__ __forceinline__ int64_t slot_of(const LayerKv& kv, int seq, int pos, int64_t block, int head, int d) {
+  const int b = kv.table[(int64_t)seq * kv.max_blocks + pos / kv.block_tokens];
+  return (int64_t)b * block + ((int64_t)head * kv.block_tokens + pos % kv.block_tokens) * d;
+}
+__device__ __forceinline__ float inv_rms(float sum_sq, int n, float eps) {
+  return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(sum_sq, (float)n), eps)));
+}
+
+// one block per row
+__global__ void __launch_bounds__(512)
+qkv_store_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bias, const float* __restrict__ q_norm,
+                 const float* __restrict__ k_norm, QkvShape sh, LayerKv kv, RowMap rows) {
+  pdl_enter();
+  __shared__ float s1[32], s2[32];
+  const int t = blockIdx.x, nq = sh.n_head * sh.dk, nk = sh.n_kv * sh.dk, nv = sh.n_kv * sh.dv;
+  float* p = proj + (int64_t)t * ld;
+  float qs = 0.f, ks = 0.f;
+  if (bias || q_norm || k_norm) {
+    for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
+      float v = p[i];
+      if (bias) { v = __fadd_rn(v, bias[i]); p[i] = v; }  // read back below by the same thread
+      if (i < nq) qs = fmaf(v, v, qs); else ks = fmaf(v, v, ks);
+    }
+    qs = block_sum(qs, s1);
+    ks = block_sum(ks, s2);
+  }
+  const int pos = row_position(rows, t), seq = row_sequence(rows, t);
+  const float qi = q_norm ? inv_rms(qs, nq, sh.eps) : 1.f, ki = k_norm ? inv_rms(ks, nk, sh.eps) : 1.f;
+  for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
+    const float v = p[i];
+    if (i < nq) {
+      if (q_norm) p[i] = __fmul_rn(__fmul_rn(v, qi), q_norm[i]);
+    } else {
+      const int c = i - nq;
+      kv.k[slot_of(kv, seq, pos, kv.k_block, c / sh.dk, sh.dk) + c % sh.dk] = k_norm ? __fmul_rn(__fmul_rn(v, ki), k_norm[c]) : v;
+    }
+  }
+  for (int c = threadIdx.x; c < nv; c += blockDim.x) {
+    float v = p[nq + nk + c];
+    if (bias) v = __fadd_rn(v, bias[nq + nk + c]);
+    kv.v[slot_of(kv, seq, pos, kv.v_block, c / sh.dv, sh.dv) + c % sh.dv] = v;
+  }
+}
+
+__global__ void __launch_bounds__(256)
+latent_store_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w, int n, float eps, LayerKv kv, RowMap rows) {
+  pdl_enter();
+  __shared__ float sh[32];
+  const int t = blockIdx.x;
+  const float* p = proj + (int64_t)t * ld;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(p[i], p[i], ss);
+  const float inv = inv_rms(block_sum(ss, sh), n, eps);
+  float* c = kv.k + slot_of(kv, row_sequence(rows, t), row_position(rows, t), kv.k_block, 0, n);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float v = __fmul_rn(p[i], inv);
+    c[i] = w ? __fmul_rn(v, w[i]) : v;
+  }
+}
+
+__global__ void __launch_bounds__(256)
+rows_bf16_kernel(const float* __restrict__ x, int64_t ld, int n, __nv_bfloat16* __restrict__ o) {
+  pdl_enter();
+  const float* xr = x + (int64_t)blockIdx.x * ld;
+  __nv_bfloat16* orow = o + (int64_t)blockIdx.x * n;
+  if ((n & 3) == 0 && (ld & 3) == 0) {
+    for (int i = 4 * threadIdx.x; i < n; i += 4 * blockDim.x) *(uint2*)(orow + i) = pack4_bf16(*(const float4*)(xr + i));
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) orow[i] = __float2bfloat16_rn(xr[i]);
+  }
+}
+
+// ---- products per head, f32 activations ---------------------------------------------------------------------------
+// y[t][h * cols + c] = sum_r W[h * rows + r][c] x[t][h * rows + r]: a thread owns two columns and every fourth row (W is
+// read along its rows), the four partial sums are added in order.
+template <int TT>
+__global__ void __launch_bounds__(256)
+head_product_t_kernel(const uint16_t* __restrict__ w, int heads, int rows, int cols, const float* __restrict__ x, int64_t x_ld,
+                      float* __restrict__ y, int tokens) {
+  pdl_enter();
+  __shared__ float part[4][TT][128];
+  const int h = blockIdx.y, t0 = blockIdx.z * TT, cp = threadIdx.x & 63, grp = threadIdx.x >> 6;
+  const int c = blockIdx.x * 128 + 2 * cp;
+  const bool two = c + 1 < cols, one = c < cols, pair = (cols & 1) == 0;
+  float a0[TT], a1[TT];
+#pragma unroll
+  for (int j = 0; j < TT; ++j) a0[j] = a1[j] = 0.f;
+  if (one) {
+    const uint16_t* wh = w + (int64_t)h * rows * cols + c;
+    const float* xh = x + (int64_t)t0 * x_ld + (int64_t)h * rows;
+#pragma unroll 8
+    for (int r = grp; r < rows; r += 4) {
+      float w0, w1;
+      if (pair) {
+        const uint32_t u = *(const uint32_t*)(wh + (int64_t)r * cols);
+        w0 = __uint_as_float(u << 16); w1 = __uint_as_float(u & 0xffff0000u);
+      } else {
+        w0 = bf(wh[(int64_t)r * cols]); w1 = two ? bf(wh[(int64_t)r * cols + 1]) : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < TT; ++j)
+        if (t0 + j < tokens) {
+          const float xv = xh[(int64_t)j * x_ld + r];
+          a0[j] = fmaf(w0, xv, a0[j]);
+          a1[j] = fmaf(w1, xv, a1[j]);
+        }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < TT; ++j) { part[grp][j][2 * cp] = a0[j]; part[grp][j][2 * cp + 1] = a1[j]; }
+  __syncthreads();
+  for (int i = threadIdx.x; i < TT * 128; i += 256) {
+    const int j = i >> 7, k = i & 127, col = blockIdx.x * 128 + k;
+    if (t0 + j < tokens && col < cols)
+      y[(int64_t)(t0 + j) * heads * cols + (int64_t)h * cols + col] = (part[0][j][k] + part[1][j][k]) + (part[2][j][k] + part[3][j][k]);
+  }
+}
+
+// y[t][h * rows + r] = sum_c W[h * rows + r][c] x[t][h * cols + c], times the head's gate: one warp per row of W
+template <int TT>
+__global__ void __launch_bounds__(256)
+head_product_kernel(const uint16_t* __restrict__ w, int heads, int rows, int cols, const float* __restrict__ x, int64_t x_ld,
+                    float* __restrict__ y, const float* __restrict__ gate, int64_t gate_ld, int tokens) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31, row = blockIdx.x * 8 + (threadIdx.x >> 5), t0 = blockIdx.y * TT;
+  if (row >= heads * rows) return;
+  const int h = row / rows;
+  const uint16_t* wr = w + (int64_t)row * cols;
+  const float* xh = x + (int64_t)t0 * x_ld + (int64_t)h * cols;
+  float acc[TT];
+#pragma unroll
+  for (int j = 0; j < TT; ++j) acc[j] = 0.f;
+  if ((cols & 3) == 0 && (x_ld & 3) == 0) {
+#pragma unroll 4
+    for (int c = 4 * lane; c < cols; c += 128) {
+      const uint2 u = *(const uint2*)(wr + c);
+      const float w0 = __uint_as_float(u.x << 16), w1 = __uint_as_float(u.x & 0xffff0000u), w2 = __uint_as_float(u.y << 16),
+                  w3 = __uint_as_float(u.y & 0xffff0000u);
+#pragma unroll
+      for (int j = 0; j < TT; ++j)
+        if (t0 + j < tokens) {
+          const float4 v = *(const float4*)(xh + (int64_t)j * x_ld + c);
+          acc[j] = fmaf(w0, v.x, fmaf(w1, v.y, fmaf(w2, v.z, fmaf(w3, v.w, acc[j]))));
+        }
+    }
+  } else {
+    for (int c = lane; c < cols; c += 32) {
+      const float wv = bf(wr[c]);
+#pragma unroll
+      for (int j = 0; j < TT; ++j)
+        if (t0 + j < tokens) acc[j] = fmaf(wv, xh[(int64_t)j * x_ld + c], acc[j]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < TT; ++j) {
+    const float v = warp_sum(acc[j]);
+    if (lane == 0 && t0 + j < tokens) {
+      const int64_t t = t0 + j;
+      y[t * heads * rows + row] = gate ? __fmul_rn(v, sigmoid(gate[t * gate_ld + h])) : v;
+    }
+  }
+}
+
+// out[h * cols + c][r] = w[h * rows + r][c] (once per session)
+__global__ void head_transpose_kernel(const uint16_t* __restrict__ w, int rows, int cols, uint16_t* __restrict__ out) {
+  const int64_t n = (int64_t)rows * cols, base = (int64_t)blockIdx.y * n;
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x)
+    out[base + (i % cols) * rows + i / cols] = w[base + i];
+}
+
+// ---- attention --------------------------------------------------------------------------------------------------
+// The keys position pos sees, as one ascending list: the kept first tokens that lie before the window, then the window.
+struct Span {
+  int lo, nk, n;  // first position of the window, kept tokens before it, visible keys
+  __device__ __forceinline__ int at(int m) const { return m < nk ? m : lo + m - nk; }
+};
+__device__ __forceinline__ Span span_of(int pos, int window, int keep_first) {
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0, nk = min(keep_first, lo);
+  return Span{lo, nk, nk + pos - lo + 1};
+}
+
+struct KvSpan {
+  const LayerKv& kv;
+  const SpanShape& sh;
+  Span span;
+  int seq, head, pos, h0;  // kv head, the row's position, first query head
+  __device__ __forceinline__ const float* k(int m) const { return kv.k + slot_of(kv, seq, span.at(m), kv.k_block, head, sh.dk); }
+  __device__ __forceinline__ const float* v(int m) const { return kv.v + slot_of(kv, seq, span.at(m), kv.v_block, head, sh.dv); }
+  __device__ __forceinline__ float score(int g, int m, float dot) const {
+    const float s = __fmul_rn(dot, sh.scale);
+    return sh.bias ? __fadd_rn(s, sh.bias[(int64_t)(h0 + g) * sh.bias_len + min(pos - span.at(m), sh.bias_len - 1)]) : s;
+  }
+};
+
+// grid (kv head x group of at most ATT_MAX_GQA query heads, slice of the visible keys, row)
+template <int MAX_VALUE>
+__global__ void __launch_bounds__(ATT_THREADS)
+span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv kv, RowMap rows, int t0, int chunk, float* __restrict__ part) {
+  pdl_enter();
+  extern __shared__ float sm[];  // q [heads][dk] | scores [heads][chunk] or sums [P][heads][dv]
+  const int gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
+  const int head = blockIdx.x / groups, g0 = (blockIdx.x % groups) * ATT_MAX_GQA, heads = min(ATT_MAX_GQA, gq - g0);
+  const int t = t0 + blockIdx.z, split = blockIdx.y, n_split = (int)gridDim.y, h0 = head * gq + g0;
+  const int pos = row_position(rows, t);
+  const Span span = span_of(pos, sh.window, sh.keep_first);
+  const int s0 = split * chunk, s1 = min(span.n, s0 + chunk);
+  if (s0 >= span.n) return;
+  float* sq = sm;
+  float* sc = sq + heads * sh.dk;
+  for (int i = threadIdx.x; i < heads * sh.dk; i += ATT_THREADS) sq[i] = q[(int64_t)t * q_ld + (int64_t)h0 * sh.dk + i];
+  __syncthreads();
+  // records: [row of the pass][query head][slice][dv + 2]; a group's heads follow each other n_split records apart
+  float* rec = part + (((int64_t)blockIdx.z * sh.n_kv * groups + blockIdx.x) * n_split + split) * ATT_MAX_GQA * (sh.dv + 2);
+  attend_slice<MAX_VALUE>(KvSpan{kv, sh, span, row_sequence(rows, t), head, pos, h0}, sq, sc, rec, s0, s1, chunk, sh.dk, sh.dv, heads);
+}
+
+// grid (query head, row): merges a head's slices (at most 32) and applies the element gate
+__global__ void __launch_bounds__(128)
+span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, int t0, int chunk, int n_split, float* __restrict__ out,
+                    __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate, int64_t gate_ld) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31, h = blockIdx.x, t = t0 + blockIdx.y;
+  const int gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
+  const int bx = (h / gq) * groups + (h % gq) / ATT_MAX_GQA, g = (h % gq) % ATT_MAX_GQA;
+  const int used = (span_of(row_position(rows, t), sh.window, sh.keep_first).n + chunk - 1) / chunk;
+  const int64_t stride = (int64_t)ATT_MAX_GQA * (sh.dv + 2);
+  const float* base = part + ((int64_t)blockIdx.y * sh.n_kv * groups + bx) * n_split * stride + g * (sh.dv + 2);
+  const float ms = lane < used ? base[lane * stride + sh.dv] : -CUDART_INF_F;
+  const float m = warp_max(ms);
+  const float e = lane < used ? expf(ms - m) : 0.f;
+  const float l = warp_sum(lane < used ? base[lane * stride + sh.dv + 1] * e : 0.f);
+  for (int i0 = 0; i0 < sh.dv; i0 += 128) {
+    const int i = i0 + threadIdx.x;
+    const bool live = i < sh.dv;
+    float acc = 0.f;
+    for (int sp = 0; sp < used; sp += 4) {
+      float v[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[j] = (live && sp + j < used) ? base[(sp + j) * stride + i] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc = fmaf(v[j], __shfl_sync(~0u, e, (sp + j) & 31), acc);  // a slice beyond `used` has value 0 and weight 0
+    }
+    if (live) {
+      float r = __fdiv_rn(acc, l);
+      const int64_t o = (int64_t)h * sh.dv + i;
+      if (gate) r = __fmul_rn(r, sigmoid(gate[(int64_t)t * gate_ld + o]));
+      if (out) out[(int64_t)t * sh.n_head * sh.dv + o] = r;
+      if (out16) out16[(int64_t)t * sh.n_head * sh.dv + o] = __float2bfloat16_rn(r);
+    }
+  }
+}
+
+// ---- prompt chunks on the tensor cores ------------------------------------------------------------------------------
+// Rows of ONE sequence at consecutive positions.  A block takes one kv head and 64 (row, query head) pairs in row-major
+// order -- all query heads of a kv head share its keys, so any ratio of heads fills the tile (one latent for every head
+// included) -- and walks the keys that any of its rows sees, 64 at a time.  Queries (rescaled per pair by a power of two),
+// keys, values and the exponentials are rounded to binary16 operands; scores and sums are m16n8k16 MMAs with f32
+// accumulators; scale, distance bias, mask, maxima, exponentials and their sums are f32.
+// Sixteen pairs belong to NS warps: each scores 64 / NS of the keys and owns 8 ND of the value dimensions.
+constexpr int CH = 64;
+__device__ __forceinline__ uint32_t pack_h2(float lo, float hi) {
+  const __half2 h = __floats2half2_rn(lo, hi);
+  return *(const uint32_t*)&h;
+}
+__device__ __forceinline__ float sat16(float v) { return fminf(fmaxf(v, -65504.f), 65504.f); }
+__device__ __forceinline__ void mma_f16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], const __half* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
+}
+__device__ __forceinline__ void ldm4_t(uint32_t (&r)[4], const __half* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
+}
+
+struct MmaLayout {  // halves; widths are multiples of 16, so a pitch is an odd number of 16-byte units
+  int kw, vw, qp, kp, vp;
+  bool shared;  // values are the keys
+};
+inline __host__ __device__ MmaLayout mma_layout(int dk, int dv, int nd, int ns, bool shared) {
+  MmaLayout L;
+  L.kw = (dk + 15) / 16 * 16;
+  L.vw = 8 * nd * ns;
+  L.shared = shared;
+  L.qp = L.kw + 8;
+  L.kp = (shared && L.vw > L.kw ? L.vw : L.kw) + 8;
+  L.vp = shared ? L.kp : L.vw + 8;
+  return L;
+}
+inline __host__ __device__ size_t mma_smem(const MmaLayout& L, int ns) {
+  return ((size_t)64 * L.qp + (size_t)CH * L.kp + (L.shared ? 0 : (size_t)CH * L.vp) + (ns > 1 ? 64 * (CH + 8) : 0)) * 2;
+}
+
+template <int ND, int NS>
+__global__ void __launch_bounds__(128 * NS)
+span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv kv, RowMap rows, int t0, int tokens, float* __restrict__ out,
+                __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate, int64_t gate_ld) {
+  pdl_enter();
+  constexpr int THR = 128 * NS, NT = CH / 8 / NS;  // score tiles of eight keys per warp
+  static_assert(NT % 2 == 0, "keys are loaded sixteen at a time");
+  extern __shared__ __align__(16) unsigned char raw[];
+  const MmaLayout L = mma_layout(sh.dk, sh.dv, ND, NS, kv.k == kv.v);
+  __half* sq = (__half*)raw;
+  __half* sk = sq + 64 * L.qp;
+  __half* sv = L.shared ? sk : sk + CH * L.kp;
+  __half* sp = sk + CH * L.kp + (L.shared ? 0 : CH * L.vp);  // exponentials, NS > 1
+  __shared__ float s_scale[64], s_red[NS][64];
+  __shared__ int64_t s_k[2][CH], s_v[2][CH];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+  const int rw = warp & 3, ns = warp >> 2;  // rows 16 rw .., key and value share ns
+  const int head = blockIdx.y, gq = sh.n_head / sh.n_kv, pairs = tokens * gq, pair0 = blockIdx.x * 64;
+  const int seq = row_sequence(rows, t0), p_first = row_position(rows, t0);
+  const int pa = p_first + pair0 / gq, pb = p_first + min(pairs - 1, pair0 + 63) / gq;  // positions of the tile's rows
+  const int lo = sh.window > 0 ? max(0, pa - sh.window + 1) : 0, nk = min(sh.keep_first, lo), n_keys = nk + pb - lo + 1;
+
+  auto offsets = [&](int c, int buf) {  // where the keys of chunk c lie
+    if (tid < CH) {
+      const int m = c * CH + tid;
+      int64_t ko = -1, vo = -1;
+      if (m < n_keys) {
+        const int j = m < nk ? m : lo + m - nk;
+        ko = slot_of(kv, seq, j, kv.k_block, head, sh.dk);
+        vo = slot_of(kv, seq, j, kv.v_block, head, sh.dv);
+      }
+      s_k[buf][tid] = ko;
+      s_v[buf][tid] = vo;
+    }
+  };
+  // queries: a warp per pair; the power of two that brings the largest magnitude into [2^9, 2^10)
+  for (int r = warp; r < 64; r += 4 * NS) {
+    const int p = pair0 + r;
+    const bool live = p < pairs;
+    const float* src = q + (int64_t)(t0 + (live ? p / gq : 0)) * q_ld + (int64_t)(head * gq + (live ? p % gq : 0)) * sh.dk;
+    float m = 0.f;
+    if (live) for (int i = lane; i < sh.dk; i += 32) m = fmaxf(m, fabsf(src[i]));
+    m = warp_max(m);
+    const int be = (int)((__float_as_uint(m) >> 23) & 0xff);
+    const int e = (be == 0 || be == 255) ? 0 : min(126, max(-126, 136 - be));
+    const float up = __uint_as_float((uint32_t)(127 + e) << 23), down = __uint_as_float((uint32_t)(127 - e) << 23);
+    for (int i = lane; i < L.kw; i += 32) sq[r * L.qp + i] = __float2half_rn(live && i < sh.dk ? sat16(src[i] * up) : 0.f);
+    if (lane == 0) s_scale[r] = down * sh.scale;
+  }
+  // padding columns of the key and value tiles are zero and stay so
+  for (int i = tid; i < CH * (L.kp - 8 - sh.dk); i += THR) sk[(i / (L.kp - 8 - sh.dk)) * L.kp + sh.dk + i % (L.kp - 8 - sh.dk)] = __float2half_rn(0.f);
+  if (!L.shared)
+    for (int i = tid; i < CH * (L.vw - sh.dv); i += THR) sv[(i / (L.vw - sh.dv)) * L.vp + sh.dv + i % (L.vw - sh.dv)] = __float2half_rn(0.f);
+  offsets(0, 0);
+  __syncthreads();
+
+  const int r0 = 16 * rw + g, r1 = r0 + 8;
+  const int i0 = p_first + min(pair0 + r0, pairs - 1) / gq, i1 = p_first + min(pair0 + r1, pairs - 1) / gq;  // positions of this thread's rows
+  const float* b0 = sh.bias ? sh.bias + (int64_t)(head * gq + min(pair0 + r0, pairs - 1) % gq) * sh.bias_len : nullptr;
+  const float* b1 = sh.bias ? sh.bias + (int64_t)(head * gq + min(pair0 + r1, pairs - 1) % gq) * sh.bias_len : nullptr;
+  const float f0 = s_scale[r0], f1 = s_scale[r1];
+  float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
+  float o[ND][4];
+#pragma unroll
+  for (int nd = 0; nd < ND; ++nd)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) o[nd][i] = 0.f;
+
+  auto row_group = [&] {  // the NS warps of sixteen pairs
+    if constexpr (NS == 1) __syncwarp();
+    else asm volatile("bar.sync %0, %1;" ::"r"(1 + rw), "r"(32 * NS) : "memory");
+  };
+  const int chunks = (n_keys + CH - 1) / CH;
+  for (int c = 0; c < chunks; ++c) {
+    const int buf = c & 1;
+    {
+      const int kv4 = sh.dk / 4;
+      for (int i = tid; i < CH * kv4; i += THR) {
+        const int p = i / kv4, d = 4 * (i % kv4);
+        const int64_t off = s_k[buf][p];
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (off >= 0) v = *(const float4*)(kv.k + off + d);
+        *(uint2*)(sk + p * L.kp + d) = make_uint2(pack_h2(sat16(v.x), sat16(v.y)), pack_h2(sat16(v.z), sat16(v.w)));
+      }
+      if (!L.shared) {
+        const int vv4 = sh.dv / 4;
+        for (int i = tid; i < CH * vv4; i += THR) {
+          const int p = i / vv4, d = 4 * (i % vv4);
+          const int64_t off = s_v[buf][p];
+          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (off >= 0) v = *(const float4*)(kv.v + off + d);
+          *(uint2*)(sv + p * L.vp + d) = make_uint2(pack_h2(sat16(v.x), sat16(v.y)), pack_h2(sat16(v.z), sat16(v.w)));
+        }
+      }
+    }
+    __syncthreads();
+    if (c + 1 < chunks) offsets(c + 1, buf ^ 1);
+    // ---- scores of this warp's keys
+    float s[NT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[nt][i] = 0.f;
+    const __half* qa = sq + (16 * rw + (lane & 15)) * L.qp + (lane >> 4) * 8;
+    const __half* kb = sk + (ns * 8 * NT + (lane & 7) + (lane >> 4) * 8) * L.kp + ((lane >> 3) & 1) * 8;
+#pragma unroll 2
+    for (int k0 = 0; k0 < L.kw; k0 += 16) {
+      uint32_t a[4];
+      ldm4(a, qa + k0);
+#pragma unroll
+      for (int nt = 0; nt < NT; nt += 2) {
+        uint32_t b[4];
+        ldm4(b, kb + nt * 8 * L.kp + k0);
+        mma_f16(s[nt], a, b[0], b[1]);
+        mma_f16(s[nt + 1], a, b[2], b[3]);
+      }
+    }
+    float x0 = -CUDART_INF_F, x1 = -CUDART_INF_F;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int m = c * CH + ns * 8 * NT + 8 * nt + 2 * t4 + i, j = m < nk ? m : lo + m - nk;
+        const bool any = m < n_keys, kept = j < sh.keep_first || sh.window <= 0;
+        float u0 = s[nt][i] * f0, u1 = s[nt][2 + i] * f1;
+        const int d0 = i0 - j, d1 = i1 - j;
+        const bool v0 = any && d0 >= 0 && (kept || d0 < sh.window), v1 = any && d1 >= 0 && (kept || d1 < sh.window);
+        if (b0 && v0) u0 += __ldg(b0 + min(d0, sh.bias_len - 1));
+        if (b1 && v1) u1 += __ldg(b1 + min(d1, sh.bias_len - 1));
+        s[nt][i] = v0 ? u0 : -CUDART_INF_F;
+        s[nt][2 + i] = v1 ? u1 : -CUDART_INF_F;
+        x0 = fmaxf(x0, s[nt][i]);
+        x1 = fmaxf(x1, s[nt][2 + i]);
+      }
+    x0 = fmaxf(x0, __shfl_xor_sync(~0u, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(~0u, x0, 2));
+    x1 = fmaxf(x1, __shfl_xor_sync(~0u, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(~0u, x1, 2));
+    if constexpr (NS > 1) {
+      if (t4 == 0) { s_red[ns][r0] = x0; s_red[ns][r1] = x1; }
+      row_group();
+#pragma unroll
+      for (int k = 0; k < NS; ++k) { x0 = fmaxf(x0, s_red[k][r0]); x1 = fmaxf(x1, s_red[k][r1]); }
+    }
+    x0 = fmaxf(x0, m0);
+    x1 = fmaxf(x1, m1);
+    const float w0 = m0 == -CUDART_INF_F ? 0.f : expf(m0 - x0), w1 = m1 == -CUDART_INF_F ? 0.f : expf(m1 - x1);
+    m0 = x0;
+    m1 = x1;
+    l0 *= w0;
+    l1 *= w1;
+#pragma unroll
+    for (int nd = 0; nd < ND; ++nd) { o[nd][0] *= w0; o[nd][1] *= w0; o[nd][2] *= w1; o[nd][3] *= w1; }
+    uint32_t e0[NT], e1[NT];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      float e[4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        e[i] = s[nt][i] == -CUDART_INF_F ? 0.f : expf(s[nt][i] - m0);
+        e[2 + i] = s[nt][2 + i] == -CUDART_INF_F ? 0.f : expf(s[nt][2 + i] - m1);
+      }
+      e0[nt] = pack_h2(e[0], e[1]);
+      e1[nt] = pack_h2(e[2], e[3]);
+      const __half2 h0 = *(const __half2*)&e0[nt], h1 = *(const __half2*)&e1[nt];
+      l0 += __low2float(h0) + __high2float(h0);  // the sum of what the weighted sum below uses
+      l1 += __low2float(h1) + __high2float(h1);
+      if constexpr (NS > 1) {
+        *(uint32_t*)(sp + r0 * (CH + 8) + ns * 8 * NT + 8 * nt + 2 * t4) = e0[nt];
+        *(uint32_t*)(sp + r1 * (CH + 8) + ns * 8 * NT + 8 * nt + 2 * t4) = e1[nt];
+      }
+    }
+    if constexpr (NS > 1) row_group();
+    // ---- weighted values: this warp's dimensions over all keys of the chunk
+    const __half* vb = sv + (lane & 15) * L.vp + ns * 8 * ND + (lane >> 4) * 8;
+#pragma unroll
+    for (int k0 = 0; k0 < CH; k0 += 16) {
+      uint32_t a[4];
+      if constexpr (NS == 1) {
+        a[0] = e0[k0 / 8]; a[1] = e1[k0 / 8]; a[2] = e0[k0 / 8 + 1]; a[3] = e1[k0 / 8 + 1];
+      } else {
+        ldm4(a, sp + (16 * rw + (lane & 15)) * (CH + 8) + k0 + (lane >> 4) * 8);
+      }
+#pragma unroll
+      for (int nd = 0; nd < ND; nd += 2) {
+        uint32_t b[4];
+        ldm4_t(b, vb + k0 * L.vp + 8 * nd);
+        mma_f16(o[nd], a, b[0], b[1]);
+        mma_f16(o[nd + 1], a, b[2], b[3]);
+      }
+    }
+    __syncthreads();  // the next chunk overwrites the tiles
+  }
+  l0 += __shfl_xor_sync(~0u, l0, 1); l0 += __shfl_xor_sync(~0u, l0, 2);
+  l1 += __shfl_xor_sync(~0u, l1, 1); l1 += __shfl_xor_sync(~0u, l1, 2);
+  if constexpr (NS > 1) {
+    if (t4 == 0) { s_red[ns][r0] = l0; s_red[ns][r1] = l1; }
+    row_group();
+    l0 = l1 = 0.f;
+#pragma unroll
+    for (int k = 0; k < NS; ++k) { l0 += s_red[k][r0]; l1 += s_red[k][r1]; }
+  }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int p = pair0 + (half ? r1 : r0);
+    if (p >= pairs) continue;
+    const int t = t0 + p / gq, h = head * gq + p % gq;
+    const float inv = __fdiv_rn(1.0f, half ? l1 : l0);
+    const int64_t base = (int64_t)h * sh.dv;
+#pragma unroll
+    for (int nd = 0; nd < ND; ++nd) {
+      const int d = ns * 8 * ND + 8 * nd + 2 * t4;
+      if (d >= sh.dv) continue;
+      float2 v = make_float2(o[nd][2 * half] * inv, o[nd][2 * half + 1] * inv);
+      if (gate) {
+        const float2 gg = *(const float2*)(gate + (int64_t)t * gate_ld + base + d);
+        v.x *= sigmoid(gg.x);
+        v.y *= sigmoid(gg.y);
+      }
+      const int64_t at = (int64_t)t * sh.n_head * sh.dv + base + d;
+      if (out) *(float2*)(out + at) = v;
+      if (out16) *(__nv_bfloat162*)(out16 + at) = __floats2bfloat162_rn(v.x, v.y);
+    }
+  }
+}
+
+// ---- norm on a sublayer's output, residual add ------------------------------------------------------------------------
+constexpr int NORM_ADD_THREADS = 512, NORM_ADD_KEEP = 4;  // up to 8192 values of a row stay in registers
+__global__ void __launch_bounds__(NORM_ADD_THREADS)
+norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, int slices, int64_t slice_stride, const float* __restrict__ w, float eps,
+                __nv_bfloat16* __restrict__ x16, int n) {
+  pdl_enter();
+  __shared__ float sh[32];
+  float* xr = x + (int64_t)blockIdx.x * n;
+  const float* yr = y + (int64_t)blockIdx.x * n;
+  __nv_bfloat16* x16r = x16 ? x16 + (int64_t)blockIdx.x * n : nullptr;
+  if (n % 4 == 0 && n <= 4 * NORM_ADD_THREADS * NORM_ADD_KEEP) {
+    float4 keep[NORM_ADD_KEEP];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NORM_ADD_KEEP; ++k) {
+      const int i = 4 * (threadIdx.x + k * NORM_ADD_THREADS);
+      if (i < n) {
+        float4 v = *(const float4*)(yr + i);
+        for (int s = 1; s < slices; ++s) {
+          const float4 u = *(const float4*)(yr + s * slice_stride + i);
+          v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+        }
+        keep[k] = v;
+        ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+      }
+    }
+    const float inv = inv_rms(block_sum(ss, sh), n, eps);
+#pragma unroll
+    for (int k = 0; k < NORM_ADD_KEEP; ++k) {
+      const int i = 4 * (threadIdx.x + k * NORM_ADD_THREADS);
+      if (i < n) {
+        const float4 ww = *(const float4*)(w + i);
+        float4 r = *(const float4*)(xr + i);
+        r.x = __fadd_rn(r.x, __fmul_rn(__fmul_rn(keep[k].x, inv), ww.x));
+        r.y = __fadd_rn(r.y, __fmul_rn(__fmul_rn(keep[k].y, inv), ww.y));
+        r.z = __fadd_rn(r.z, __fmul_rn(__fmul_rn(keep[k].z, inv), ww.z));
+        r.w = __fadd_rn(r.w, __fmul_rn(__fmul_rn(keep[k].w, inv), ww.w));
+        *(float4*)(xr + i) = r;
+        if (x16r) *(uint2*)(x16r + i) = pack4_bf16(r);
+      }
+    }
+    return;
+  }
+  auto value = [&](int i) {
+    float v = yr[i];
+    for (int s = 1; s < slices; ++s) v += yr[s * slice_stride + i];
+    return v;
+  };
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = value(i); ss = fmaf(v, v, ss); }
+  const float inv = inv_rms(block_sum(ss, sh), n, eps);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float r = __fadd_rn(xr[i], __fmul_rn(__fmul_rn(value(i), inv), w[i]));
+    xr[i] = r;
+    if (x16r) x16r[i] = __float2bfloat16_rn(r);
+  }
+}
+
+// ---- clamped gated unit -------------------------------------------------------------------------------------------
+__device__ __forceinline__ float clamped_glu(float a, float b, const GluShape& sh) {
+  a = fminf(a, sh.limit);
+  b = fminf(fmaxf(b, -sh.limit), sh.limit);
+  return __fmul_rn(__fmul_rn(a, sigmoid(__fmul_rn(sh.alpha, a))), __fadd_rn(b, sh.shift));
+}
+__global__ void __launch_bounds__(256)
+clamped_glu_kernel(const float* __restrict__ gu, GluShape sh, float* __restrict__ out, __nv_bfloat16* __restrict__ out16, int tokens) {
+  pdl_enter();
+  const int64_t step = (int64_t)gridDim.x * blockDim.x, first = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (sh.n % 4 == 0) {
+    const int n4 = sh.n / 4;
+    for (int64_t i = first; i < (int64_t)tokens * n4; i += step) {
+      const int64_t t = i / n4, c = 4 * (i % n4);
+      const float4 a = *(const float4*)(gu + t * 2 * sh.n + c), b = *(const float4*)(gu + t * 2 * sh.n + sh.n + c);
+      const float4 r = make_float4(clamped_glu(a.x, b.x, sh), clamped_glu(a.y, b.y, sh), clamped_glu(a.z, b.z, sh), clamped_glu(a.w, b.w, sh));
+      if (out) *(float4*)(out + t * sh.n + c) = r;
+      if (out16) *(uint2*)(out16 + t * sh.n + c) = pack4_bf16(r);
+    }
+    return;
+  }
+  for (int64_t i = first; i < (int64_t)tokens * sh.n; i += step) {
+    const int64_t t = i / sh.n, c = i % sh.n;
+    const float r = clamped_glu(gu[t * 2 * sh.n + c], gu[t * 2 * sh.n + sh.n + c], sh);
+    if (out) out[i] = r;
+    if (out16) out16[i] = __float2bfloat16_rn(r);
+  }
+}
+
+// ---- launch shapes of the attention kernels ---------------------------------------------------------------------------
+constexpr int MAX_VALUE = 512;
+int span_visible(const SpanShape& sh) {
+  return sh.window > 0 ? (int)std::min<int64_t>(sh.n_ctx, (int64_t)sh.window + sh.keep_first) : sh.n_ctx;
+}
+int span_chunk(const SpanShape& sh) { return std::max(32, (span_visible(sh) + 31) / 32); }
+int span_splits(const SpanShape& sh) { return (span_visible(sh) + span_chunk(sh) - 1) / span_chunk(sh); }
+size_t span_row_floats(const SpanShape& sh) {
+  const size_t gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
+  return sh.n_kv * groups * span_splits(sh) * ATT_MAX_GQA * (size_t)(sh.dv + 2);
+}
+size_t span_smem(const SpanShape& sh) {
+  const size_t heads = std::min(ATT_MAX_GQA, sh.n_head / sh.n_kv), P = std::max(1, ATT_THREADS / sh.dv);
+  return (heads * sh.dk + std::max(heads * span_chunk(sh), P * heads * sh.dv)) * sizeof(float);
+}
+constexpr size_t SCRATCH_FLOATS = 16u << 20;
+int span_rows_per_pass(const SpanShape& sh) { return (int)std::min<size_t>(512, std::max<size_t>(1, SCRATCH_FLOATS / span_row_floats(sh))); }
+
+typedef void (*MmaKernel)(const float*, int64_t, SpanShape, LayerKv, RowMap, int, int, float*, __nv_bfloat16*, const float*, int64_t);
+// the smallest instantiation that covers the value dimensions
+MmaKernel mma_kernel(int dv, int* nd, int* ns) {
+#define LLR_SPAN(N, S) if (dv <= 8 * N * S) { *nd = N; *ns = S; return span_mma_kernel<N, S>; }
+  LLR_SPAN(4, 1) LLR_SPAN(8, 1) LLR_SPAN(12, 1) LLR_SPAN(16, 1) LLR_SPAN(12, 2) LLR_SPAN(16, 2) LLR_SPAN(12, 4) LLR_SPAN(16, 4)
+#undef LLR_SPAN
+  return nullptr;
+}
+
+}  // namespace
+
+cudaError_t launch_embed(const void* table, const void* pos_table, const int* ids, const RowMap& rows, float scale, float* x, void* x16,
+                         int tokens, int n, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  return launch_walk(embed_kernel, dim3(tokens), dim3(256), 0, s, (const uint16_t*)table, (const uint16_t*)pos_table, ids, rows, scale, x,
+                     (__nv_bfloat16*)x16, n);
+}
+
+cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh,
+                             const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  return launch_walk(qkv_store_kernel, dim3(tokens), dim3(512), 0, s, proj, ld, bias, q_norm, k_norm, sh, kv, rows);
+}
+
+cudaError_t launch_latent_store(const float* proj, int ld, const float* w, int n, float eps, const LayerKv& kv, const RowMap& rows, int tokens,
+                                cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  return launch_walk(latent_store_kernel, dim3(tokens), dim3(256), 0, s, proj, ld, w, n, eps, kv, rows);
+}
+
+cudaError_t launch_rows_bf16(const float* x, int64_t ld, int n, void* out16, int tokens, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  return launch_walk(rows_bf16_kernel, dim3(tokens), dim3(256), 0, s, x, ld, n, (__nv_bfloat16*)out16);
+}
+
+cudaError_t launch_head_product_t(const void* w, int heads, int rows, int cols, const float* x, int64_t x_ld, float* y, int tokens, cudaStream_t s,
+                                  uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  if (tokens == 1)
+    return launch_walk(head_product_t_kernel<1>, dim3((cols + 127) / 128, heads, 1), dim3(256), 0, s, (const uint16_t*)w, heads, rows, cols, x, x_ld, y, tokens);
+  return launch_walk(head_product_t_kernel<8>, dim3((cols + 127) / 128, heads, (tokens + 7) / 8), dim3(256), 0, s, (const uint16_t*)w, heads, rows, cols, x,
+                     x_ld, y, tokens);
+}
+
+cudaError_t launch_head_product(const void* w, int heads, int rows, int cols, const float* x, int64_t x_ld, float* y, const float* gate,
+                                int64_t gate_ld, int tokens, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  if (tokens == 1)
+    return launch_walk(head_product_kernel<1>, dim3((heads * rows + 7) / 8, 1), dim3(256), 0, s, (const uint16_t*)w, heads, rows, cols, x, x_ld, y, gate,
+                       gate_ld, tokens);
+  return launch_walk(head_product_kernel<8>, dim3((heads * rows + 7) / 8, (tokens + 7) / 8), dim3(256), 0, s, (const uint16_t*)w, heads, rows, cols, x, x_ld,
+                     y, gate, gate_ld, tokens);
+}
+
+cudaError_t launch_head_transpose(const void* w, int heads, int rows, int cols, void* out, cudaStream_t s, uint64_t* launches) {
+  if (launches) ++*launches;
+  head_transpose_kernel<<<dim3((unsigned)std::min<int64_t>(((int64_t)rows * cols + 255) / 256, 256), heads), 256, 0, s>>>((const uint16_t*)w, rows, cols,
+                                                                                                                     (uint16_t*)out);
+  return cudaGetLastError();
+}
+
+bool span_supported(const SpanShape& sh) {
+  return sh.n_head > 0 && sh.n_kv > 0 && sh.n_head % sh.n_kv == 0 && sh.dk > 0 && sh.dv > 0 && sh.dv <= MAX_VALUE && sh.dk <= 1024 && sh.n_head <= 4096 &&
+         span_smem(sh) <= 200 * 1024;
+}
+size_t span_scratch_floats(const SpanShape& sh) { return (size_t)span_rows_per_pass(sh) * span_row_floats(sh); }
+
+cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape& sh, const LayerKv& kv, const RowMap& rows, int t0, int tokens,
+                                  float* out, void* out16, const float* gate, int64_t gate_ld, float* scratch, bool tensor_cores, bool one_sequence,
+                                  cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (!span_supported(sh)) return cudaErrorInvalidValue;
+  const int gq = sh.n_head / sh.n_kv;
+  if (tensor_cores && one_sequence && sh.dk % 8 == 0 && sh.dv % 8 == 0 && q_ld % 4 == 0 && gate_ld % 2 == 0 && ((uintptr_t)gate & 7) == 0) {
+    int nd = 0, ns = 0;
+    MmaKernel kern = mma_kernel(sh.dv, &nd, &ns);
+    const size_t smem = kern ? mma_smem(mma_layout(sh.dk, sh.dv, nd, ns, kv.k == kv.v), ns) : 0;
+    if (kern && smem <= 200 * 1024) {
+      if (smem > 40 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+      }
+      if (launches) ++*launches;
+      return launch_walk(kern, dim3((unsigned)(((int64_t)tokens * gq + 63) / 64), sh.n_kv), dim3(128 * ns), smem, s, q, q_ld, sh, kv, rows, t0, tokens, out,
+                         (__nv_bfloat16*)out16, gate, gate_ld);
+    }
+  }
+  const int groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA, chunk = span_chunk(sh), splits = span_splits(sh), per = span_rows_per_pass(sh);
+  const size_t smem = span_smem(sh);
+  auto kern = sh.dv <= ATT_THREADS ? span_partial_kernel<ATT_THREADS> : span_partial_kernel<MAX_VALUE>;
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+  }
+  for (int r = 0; r < tokens; r += per) {
+    const int n = std::min(per, tokens - r);
+    if (launches) *launches += 2;
+    cudaError_t e = launch_walk(kern, dim3(sh.n_kv * groups, splits, n), dim3(ATT_THREADS), smem, s, q, q_ld, sh, kv, rows, t0 + r, chunk, scratch);
+    if (e != cudaSuccess) return e;
+    e = launch_walk(span_combine_kernel, dim3(sh.n_head, n), dim3(128), 0, s, (const float*)scratch, sh, rows, t0 + r, chunk, splits, out,
+                    (__nv_bfloat16*)out16, gate, gate_ld);
+    if (e != cudaSuccess) return e;
+  }
+  return cudaSuccess;
+}
+
+cudaError_t launch_norm_add(float* x, const float* y, int slices, int64_t slice_stride, const float* w, float eps, void* x16, int tokens, int n,
+                            cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  return launch_walk(norm_add_kernel, dim3(tokens), dim3(NORM_ADD_THREADS), 0, s, x, y, slices, slice_stride, w, eps, (__nv_bfloat16*)x16, n);
+}
+
+cudaError_t launch_clamped_glu(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  const int64_t n = (int64_t)tokens * sh.n / (sh.n % 4 == 0 ? 4 : 1);
+  return launch_walk(clamped_glu_kernel, dim3((unsigned)std::max<int64_t>(1, std::min<int64_t>((n + 255) / 256, 148 * 8))), dim3(256), 0, s, gu, sh, out,
+                     (__nv_bfloat16*)out16, tokens);
+}
+
+}  // namespace llr

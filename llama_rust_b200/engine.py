@@ -23,7 +23,7 @@ ERR_OOM = 7
 class EngineCfg:
     """EngineCfg (engine.rs:253-294), the knobs that concern batch formation."""
     max_seqs: int = 4
-    prefill_chunk: int = 0      # prompt tokens per sequence per step; 0: the rest of the prompt
+    prefill_chunk: int = 0      # prompt tokens per sequence per step; 0: the rest of the prompt, as far as the batch has room
     eos: int | None = None
     decode_first: bool = False  # hold prompt chunks while any sequence decodes
 
@@ -187,11 +187,15 @@ class Engine:
     def _prefill_and_replay(self) -> int:
         hold = self.cfg.decode_first and any(self._is_decode(i) for i in range(len(self.slots)))
         jobs = []
+        replays = [i for i, s in enumerate(self.slots) if not self._is_prefill(i) and self._is_decode(i) and s.replay < len(s.generated)]
+        room = self.s.max_batch - len(replays)  # rows of the batch left for prompt chunks
         for i, s in enumerate(self.slots):
             if self._is_prefill(i):
-                if not hold:
-                    jobs.append((i, self.s.prompt_suffix(s.prompt, i, self.cfg.prefill_chunk), "prompt"))
-            elif self._is_decode(i) and s.replay < len(s.generated):
+                if not hold and room > 0:
+                    chunk = min(self.cfg.prefill_chunk, room) if self.cfg.prefill_chunk else room
+                    jobs.append((i, self.s.prompt_suffix(s.prompt, i, chunk), "prompt"))
+                    room -= len(jobs[-1][1])
+            elif i in replays:
                 jobs.append((i, [s.generated[s.replay]], "replay"))
         return self._forward(jobs) if jobs else 0
 

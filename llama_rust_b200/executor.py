@@ -145,11 +145,12 @@ class Session:
         model = _lib.LlamaModel(c, token_embd._h, output._h if output is not None else None, norm(output_norm), arr)
         h = C.c_void_p()
         executor._check(lib().llr_session_create_paged(executor._h, C.byref(model), n_seq, kv_blocks, block_tokens, C.byref(h)))
-        self._h = h.value
-        self.n_seq = n_seq
-        self.n_vocab = int(cfg["n_vocab"])
         self._keep = []
-        self._model = (token_embd, output, layers)  # the device reads these matrices for as long as the session lives
+        self._adopt(h.value, n_seq, int(cfg["n_vocab"]), int(cfg["n_embd"]), (token_embd, output, layers))
+
+    def _adopt(self, handle: int, n_seq: int, n_vocab: int, n_embd: int, model) -> None:
+        self._h, self.n_seq, self.n_vocab, self.n_embd = handle, n_seq, n_vocab, n_embd
+        self._model = model  # the device reads these matrices for as long as the session lives
         self._ids = [[] for _ in range(n_seq)]  # token ids whose keys and values each sequence's cache holds
 
     def prefill(self, tokens, want_logits: bool = False):
@@ -180,6 +181,56 @@ class Session:
         for q, t in groups:
             self._ids[q].extend(int(v) for v in t)
         return nxt, lg
+
+    @property
+    def max_batch(self) -> int:
+        """Most rows one batch may have."""
+        n = C.c_size_t()
+        self._exec._check(lib().llr_session_max_batch(self._h, C.byref(n)))
+        return n.value
+
+    def batch_rows(self, groups, want):
+        """One ragged batch as in batch(); `want` names rows of it (indices into the groups' tokens laid end to end).
+        Returns their logits [len(want), n_vocab]."""
+        seqs = np.array([g[0] for g in groups], np.uint32)
+        counts = np.array([len(g[1]) for g in groups], np.uint32)
+        toks = np.ascontiguousarray(np.concatenate([np.asarray(g[1], np.int32) for g in groups]), np.int32)
+        w = np.array(want, np.uint32)
+        out = np.empty((w.size, self.n_vocab), np.float32)
+        self._exec._check(lib().llr_session_batch_rows(self._h, len(groups), seqs.ctypes.data, counts.ctypes.data, toks.ctypes.data,
+                                                       w.size, w.ctypes.data, out.ctypes.data))
+        for q, t in groups:
+            self._ids[q].extend(int(v) for v in t)
+        return out
+
+    def forward(self, groups, want):
+        """Appends groups of any length, in as many batches as the session's batch size needs.  groups: (sequence index,
+        token ids); want: per group the places among its tokens whose logits are asked for.  Returns them
+        [sum of wants, n_vocab], in the order of the groups and of each group's `want`."""
+        out = np.empty((sum(len(w) for w in want), self.n_vocab), np.float32)
+        base = np.cumsum([0] + [len(w) for w in want])
+        done, cap = [0] * len(groups), self.max_batch
+        while any(done[g] < len(t) for g, (_, t) in enumerate(groups)):
+            part, rows, places, room = [], [], [], cap
+            for g, (q, t) in enumerate(groups):
+                n = min(room, len(t) - done[g])
+                if n <= 0:
+                    continue
+                for k, p in enumerate(want[g]):
+                    if done[g] <= p < done[g] + n:
+                        rows.append(cap - room + p - done[g])
+                        places.append(base[g] + k)
+                part.append((q, t[done[g]:done[g] + n]))
+                done[g] += n
+                room -= n
+            out[places] = self.batch_rows(part, rows)
+        return out
+
+    def residual(self, n_rows: int) -> np.ndarray:
+        """The residual stream of the last batch's first rows."""
+        out = np.empty((n_rows, self.n_embd), np.float32)
+        self._exec._check(lib().llr_session_residual(self._h, n_rows, out.ctypes.data, out.size))
+        return out
 
     def cached_ids(self, seq: int = 0) -> list:
         return list(self._ids[seq])
@@ -245,6 +296,52 @@ class Session:
             self.free()
         except Exception:
             pass
+
+
+MIXER_ATTENTION, MIXER_LATENT = 0, 1
+GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
+
+
+class DecoderSession(Session):
+    """A session of a decoder described layer by layer (llr_session_create_decoder): everything a Session does."""
+
+    def __init__(self, executor: "Executor", cfg: dict, token_embd: Matrix, layers, output_norm, pos_embd: Matrix | None = None,
+                 output: Matrix | None = None, n_seq: int = 1, kv_blocks: int = 0, block_tokens: int = 16):
+        """cfg: n_embd, n_vocab, n_ctx, norm_eps, embd_scale.  layers: per layer a dict
+        mixer: kind, n_head, dim, vdim, scale, in, out (Matrix) and, where the mixer has them, n_head_kv, kv_rank, window,
+          keep_first, kv_from, gate, up_k, up_v (Matrix), in_bias, q_norm, k_norm, kv_norm (arrays), rel (array
+          [n_bucket, n_head]) and bias_max;
+        mlp: None, or n_ff, limit, alpha, shift, gate_up, down (Matrix);
+        mixer_norm, mlp_norm: arrays of n_embd."""
+        self._exec = executor
+        self._h = None
+        keep = []
+
+        def host(v):
+            if v is None:
+                return None
+            keep.append(np.ascontiguousarray(v, np.float32))
+            return keep[-1].ctypes.data
+
+        def dev(m):
+            return m._h if m is not None else None
+        arr = (_lib.DecoderLayer * len(layers))()
+        for i, L in enumerate(layers):
+            m, f = L["mixer"], L.get("mlp")
+            rel = m.get("rel")
+            arr[i].mixer = _lib.Mixer(
+                m["kind"], m["n_head"], m.get("n_head_kv", 0), m["dim"], m["vdim"], m.get("kv_rank", 0), m.get("window", 0),
+                m.get("keep_first", 0), m.get("kv_from", -1), m.get("gate", GATE_NONE), float(m["scale"]),
+                0 if rel is None else len(rel), m.get("bias_max", 0), dev(m["in"]), dev(m.get("up_k")), dev(m.get("up_v")), dev(m["out"]),
+                host(m.get("in_bias")), host(m.get("q_norm")), host(m.get("k_norm")), host(m.get("kv_norm")), host(rel))
+            if f is not None:
+                arr[i].mlp = _lib.Mlp(f["n_ff"], f["limit"], f["alpha"], f["shift"], dev(f["gate_up"]), dev(f["down"]))
+            arr[i].mixer_norm, arr[i].mlp_norm = host(L["mixer_norm"]), host(L.get("mlp_norm"))
+        model = _lib.DecoderModel(len(layers), cfg["n_embd"], cfg["n_vocab"], cfg["n_ctx"], cfg["norm_eps"], cfg["embd_scale"],
+                                  dev(token_embd), dev(pos_embd), dev(output), host(output_norm), arr)
+        h = C.c_void_p()
+        executor._check(lib().llr_session_create_decoder(executor._h, C.byref(model), n_seq, kv_blocks, block_tokens, C.byref(h)))
+        self._adopt(h.value, n_seq, cfg["n_vocab"], cfg["n_embd"], (token_embd, pos_embd, output, layers))
 
 
 MOVE_WEIGHTS, DISPATCH_ACTIVATIONS = 0, 1

@@ -16,7 +16,8 @@ def _next(tokens):
 
 
 class FakeSession:
-    """The part of Session the Engine uses: batch, seq_position, seq_reset, prompt_suffix; blocks of `block` positions."""
+    """The part of Session the Engine uses: batch, max_batch, seq_position, seq_reset, prompt_suffix; blocks of `block` positions."""
+    max_batch = 512
 
     def __init__(self, n_seq, kv_blocks, block=2):
         self.n_seq, self.free, self.block = n_seq, kv_blocks, block

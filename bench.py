@@ -22,7 +22,8 @@ measured HBM peak; `cpu_baseline` is the CPU oracle (AVX2 row kernels, reference
 on a bounded sample of the same sweep.  `configs` holds the other benchmark configurations (1: the
 single Q8_0 product; every format's decode kernel on one large matrix; 4: the chunk GEMM; 5: the
 routed-expert layer, at N > 1 expert-parallel over peer stores beside the NCCL all-to-all form;
-3: the walk on the device).  `--case gemv|moe|session` runs one small case for profiling.
+3: the walk on the device).  `--case gemv|moe|session` runs one small case for profiling;
+`--case decoder` times layered decoders beside the Llama walk at equal sizes.
 """
 from __future__ import annotations
 
@@ -771,14 +772,121 @@ def check_sharded(ex, sharded, offs, shape_of, xin, phase_of, M, world, rank, sp
             "how": "first layers of the sharded program vs the same products unsharded on each rank's own GPU, all rows, uint32 compare"}
 
 
+DECODER_SIZES = {  # layer sizes of real models: width, query heads, key/value heads, head size, ff, latent size
+    "1b": dict(width=2048, heads=16, kv_heads=8, dim=128, ff=8192, rank=512, vocab=32000),
+    "8b": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=14336, rank=512, vocab=32000),
+    "wide": dict(width=6144, heads=48, kv_heads=12, dim=128, ff=16384, rank=512, vocab=32000),
+}
+
+
+def layered_session(ex, z, kinds, n_ctx, window, n_seq=1):
+    """A Nagolix-shaped session with random BF16 weights: one layer per entry of `kinds` ("attention", "latent", "shared":
+    a latent layer that reads the cache of the latent layer before it)."""
+    from llama_rust_b200 import DTYPES, DecoderSession
+    from llama_rust_b200.executor import GATE_ELEMENT, GATE_HEAD, MIXER_ATTENTION, MIXER_LATENT
+    BF16 = DTYPES["BF16"]
+    W, H, G, d, R = z["width"], z["heads"], z["kv_heads"], z["dim"], z["rank"]
+    seed = [100]
+
+    def mat(rows, cols):
+        seed[0] += 1
+        return ex.synth(BF16, rows, cols, seed[0])
+    ones, rng = np.ones(W, np.float32), np.random.default_rng(1)
+    layers, source = [], -1
+    for i, kind in enumerate(kinds):
+        if kind == "attention":
+            m = dict(kind=MIXER_ATTENTION, n_head=H, n_head_kv=G, dim=d, vdim=d, scale=d ** -0.5, window=window, keep_first=4, gate=GATE_ELEMENT,
+                     rel=rng.standard_normal((32, H)).astype(np.float32), bias_max=128, in_bias=np.zeros((H + 2 * G) * d, np.float32),
+                     q_norm=np.ones(H * d, np.float32), k_norm=np.ones(G * d, np.float32), out=mat(W, H * d))
+            m["in"] = mat((2 * H + 2 * G) * d, W)
+        else:
+            own = kind == "latent"
+            m = dict(kind=MIXER_LATENT, n_head=H, dim=d, vdim=d, kv_rank=R, scale=d ** -0.5, kv_from=-1 if own else source, window=window, gate=GATE_HEAD,
+                     up_k=mat(H * d, R), up_v=mat(H * d, R), kv_norm=np.ones(R, np.float32) if own else None, out=mat(W, H * d))
+            m["in"] = mat(H * d + (R if own else 0) + H, W)
+            source = i if own else source
+        layers.append(dict(mixer=m, mixer_norm=ones, mlp_norm=ones,
+                           mlp=dict(n_ff=z["ff"], limit=7.0, alpha=1.702, shift=1.0, gate_up=mat(2 * z["ff"], W), down=mat(W, z["ff"]))))
+    return DecoderSession(ex, dict(n_embd=W, n_vocab=z["vocab"], n_ctx=n_ctx, norm_eps=1e-6, embd_scale=1.0), mat(z["vocab"], W), layers, ones,
+                          pos_embd=mat(n_ctx, W), n_seq=n_seq)
+
+
+def llama_session(ex, z, n_layer, n_ctx, n_seq=1):
+    """The Llama walk at the same sizes, BF16 weights."""
+    from llama_rust_b200 import DTYPES, Session
+    BF16, W, H, G, d = DTYPES["BF16"], z["width"], z["heads"], z["kv_heads"], z["dim"]
+    shapes = dict(attn_q=(H * d, W), attn_k=(G * d, W), attn_v=(G * d, W), attn_output=(W, H * d), ffn_gate=(z["ff"], W), ffn_up=(z["ff"], W),
+                  ffn_down=(W, z["ff"]))
+    layers = [{k: ex.synth(BF16, r, c, 500 + 10 * li + j) for j, (k, (r, c)) in enumerate(shapes.items())} for li in range(n_layer)]
+    cfg = dict(n_layer=n_layer, n_embd=W, n_head=H, n_head_kv=G, head_dim=d, n_ff=z["ff"], n_vocab=z["vocab"], n_ctx=n_ctx)
+    return Session(ex, cfg, ex.synth(BF16, z["vocab"], W, 1), layers, output=ex.synth(BF16, z["vocab"], W, 2), n_seq=n_seq)
+
+
+def decoder_case(args):
+    """--case decoder: prefill and decode of layered decoders beside the Llama walk at equal sizes, random BF16 weights.
+    Prompt tokens go in chunks of 512; decode starts behind the prompt.  Wall time of the session calls (host token ids in
+    and out, one synchronization per call).  Layer weights exceed L2 (126 MB), so nothing is flushed between steps."""
+    import torch
+    from llama_rust_b200 import Executor, synth
+    runs = {"llama": None, "attention": ["attention"] * args.layers, "latent": ["latent"] * args.layers,
+            "mixed": (["latent", "attention", "attention", "shared"] * args.layers)[:args.layers]}
+    if args.model:
+        runs = {args.model: runs[args.model]}
+    out = {"case": "decoder", "layers": args.layers, "prompt": args.prompt, "gen": args.gen, "window": args.window, "data": "synthetic", "dtype": "bf16", "sizes": {}}
+    clocks = ClockSampler(torch.cuda.current_device())
+    clocks.start()
+    for name in (args.size.split(",") if args.size else DECODER_SIZES):
+        z, res = DECODER_SIZES[name], {}
+        n_ctx = max(args.ctx, args.prompt + args.gen + 8)
+        for what, kinds in runs.items():
+            ex = Executor(0)
+            if args.path is not None:
+                ex.set_path(args.path)
+            s = llama_session(ex, z, args.layers, n_ctx, max(1, args.batch)) if kinds is None else layered_session(ex, z, kinds, n_ctx, args.window, max(1, args.batch))
+            prompt = (synth.words(7, 0, args.prompt) % np.uint64(z["vocab"])).astype(np.int32)
+            best = [1e9, 1e9]
+            for rep in range(args.reps if args.reps != 20 else 4):  # the first is the warm-up
+                s.reset()
+                t0 = time.perf_counter()
+                s.prefill(prompt)
+                t1 = time.perf_counter()
+                s.decode(args.gen)
+                t2 = time.perf_counter()
+                if rep or args.reps == 1:
+                    best = [min(best[0], t1 - t0), min(best[1], t2 - t1)]
+            r = {"prefill_ms": best[0] * 1e3, "prefill_tok_s": args.prompt / best[0], "decode_ms_per_token": best[1] / args.gen * 1e3,
+                 "decode_tok_s": args.gen / best[1]}
+            if args.batch:  # a decode batch over several sequences, each behind its own short prompt
+                s.reset()
+                groups = [(q, prompt[:32].tolist()) for q in range(args.batch)]
+                s.forward(groups, [[] for _ in groups])
+                step = [(q, [int(prompt[q])]) for q in range(args.batch)]
+                for _ in range(3):
+                    s.batch(step)
+                t0 = time.perf_counter()
+                for _ in range(8):
+                    s.batch(step)
+                r["batch_step_ms"] = (time.perf_counter() - t0) / 8 * 1e3
+            res[what] = {k: round(v, 4) for k, v in r.items()}
+            s.free()
+            ex.close()
+        out["sizes"][name] = res
+    out["clocks"] = clocks.stop()
+    print(json.dumps(out))
+
+
 def run_case(args):
     """One small case for profiling (the full sweep holds 5 GB): prints one JSON line.
       --case gemv    --dtype D --rows R --cols C --m M --reps N --copies K [--path P]   device-pointer products round-robin over K matrices
       --case moe     --tokens T                                                        the routed-expert layer of benchmark config 5 (2 warm-up + 5 timed calls)
       --case session --prompt P --gen G [--layers L] [--experts E]                     the device-resident walk on an 8B-shaped model of L layers
-                                                                                       (E routed experts per layer, two per token, instead of the dense FFN)"""
+                                                                                       (E routed experts per layer, two per token, instead of the dense FFN)
+      --case decoder --prompt P --gen G --layers L [--size S] [--model M] [--window W] [--batch B]
+                                                                                       layered decoders beside the Llama walk at equal sizes, BF16"""
     import torch
     from llama_rust_b200 import DTYPES, Executor, row_bytes as lib_row_bytes, synth
+    if args.case == "decoder":
+        return decoder_case(args)
     ex = Executor(0)
     if args.path is not None:
         ex.set_path(args.path)
@@ -844,7 +952,7 @@ def main():
     ap.add_argument("--no-configs", action="store_true", help="skip the legs for benchmark configs 1, 4 and 5")
     ap.add_argument("--mode", default="program", choices=["program", "calls"],
                     help="program: the sweep as one persistent launch; calls: one launch per matmul")
-    ap.add_argument("--case", default=None, choices=["gemv", "moe", "session"], help="run one small case instead of the sweep (for profiling)")
+    ap.add_argument("--case", default=None, choices=["gemv", "moe", "session", "decoder"], help="run one small case instead of the sweep (for profiling)")
     ap.add_argument("--dtype", default="Q4_K")
     ap.add_argument("--rows", type=int, default=65536)
     ap.add_argument("--cols", type=int, default=4096)
@@ -857,6 +965,10 @@ def main():
     ap.add_argument("--layers", type=int, default=4)
     ap.add_argument("--ctx", type=int, default=0, help="--case session: context length of the session (default: prompt + gen + 8)")
     ap.add_argument("--experts", type=int, default=0, help="--case session: routed experts per layer (0: dense FFN)")
+    ap.add_argument("--size", default=None, help="--case decoder: sizes to run, with commas (default: all)")
+    ap.add_argument("--model", default=None, choices=["llama", "attention", "latent", "mixed"], help="--case decoder: one of the models only")
+    ap.add_argument("--window", type=int, default=1024, help="--case decoder: window of the layered decoders")
+    ap.add_argument("--batch", type=int, default=0, help="--case decoder: also time decode batches over this many sequences")
     args = ap.parse_args()
     if args.case:
         return run_case(args)

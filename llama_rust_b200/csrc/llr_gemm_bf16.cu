@@ -9,15 +9,20 @@
 // rows (x16); results are f32, or bfloat16 for the product that follows, optionally multiplied by the sigmoid of a
 // per-head gate.
 //
-// One CTA computes a tile of 128 activation rows x BN weight rows: the activation rows are the MMA's M dimension (one
+// With `glu` W stacks gate | up (2 rows rows) and the results are clamped gated units: a tile then holds as many gate rows
+// as up rows, so that a thread of the epilogue has both factors of each result.
+//
+// One CTA computes a tile of 128 activation rows x bn <= BN weight rows: the activation rows are the MMA's M dimension (one
 // tensor-memory lane each), so that a thread of the epilogue holds consecutive results of one activation row and stores
 // them as vectors.  Six warps: four read the accumulators, one issues the TMA loads, one the MMAs.  Two CTAs fit an SM
 // at BN <= 128 (96 KB of stages, 128 columns of tensor memory each), so one tile's epilogue overlaps another's loads.
-// A K range may be cut into slices (gridDim.z): slice s leaves its partial sums at y + s * slice_stride and the reader
+// bn is the width, a multiple of sixteen, for which the grid's waves over the SMs cost least.  A K range may be cut into slices (gridDim.z): slice s leaves its partial sums at y + s * slice_stride and the reader
 // adds them in slice order.  Every wait is bounded.
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
+
+#include <algorithm>
 
 #include "llr_formats.cuh"
 #include "llr_kernels.cuh"
@@ -64,9 +69,9 @@ __device__ __forceinline__ bool elect_one() {
 __device__ __forceinline__ uint64_t tile_desc(uint32_t saddr) {
   return ((uint64_t)(saddr >> 4) & 0x3fffu) | (1ull << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
 }
-// kind::f16: f32 accumulator, both operands bfloat16, M = 128, N = BN
-template <int BN> __host__ __device__ constexpr uint32_t mma_desc() {
-  return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
+// kind::f16: f32 accumulator, both operands bfloat16, M = 128, N = bn
+__device__ __forceinline__ uint32_t mma_desc(int bn) {
+  return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(bn >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
 }
 
 struct Args {
@@ -75,10 +80,28 @@ struct Args {
   const float* gate;   // gate[t * gate_ld + z]: results times its sigmoid
   int64_t y_ld, gate_ld, slice_stride;
   int tokens, rows, nk, xk;  // nk: 64-column steps of the whole K range
-  int batch, slices;
+  int batch, slices, bn;
+  GluShape glu;
 };
 
-template <int BN>
+// 32 accumulator columns of this warp's 32 lanes
+__device__ __forceinline__ void load32(uint32_t taddr, uint32_t (&v)[32]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
+      "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
+        "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]),
+        "=r"(v[16]), "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]),
+        "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+      : "r"(taddr) : "memory");
+}
+__device__ __forceinline__ float glu_of(float a, float b, const GluShape& g) {
+  a = fminf(a, g.limit);
+  b = fminf(fmaxf(b, -g.limit), g.limit);
+  return a * __fdiv_rn(1.0f, 1.0f + expf(-g.alpha * a)) * (b + g.shift);
+}
+
+template <int BN, bool GLU>
 __global__ void __launch_bounds__(THREADS)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap, const Args a, int* __restrict__ err) {
   using L = Lay<BN>;
@@ -90,7 +113,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
   uint64_t* done = empty + NS;
   uint32_t* tmem_slot = (uint32_t*)(done + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int row0 = blockIdx.x * BN, tok0 = blockIdx.y * BM;
+  const int bn = a.bn, width = GLU ? bn / 2 : bn;  // results per activation row of the tile
+  const int row0 = blockIdx.x * width, tok0 = blockIdx.y * BM;
   const int z = (int)blockIdx.z / a.slices, slice = (int)blockIdx.z % a.slices;
   const int per = (a.nk + a.slices - 1) / a.slices, k0 = slice * per, k1 = min(a.nk, k0 + per);  // never empty: the launcher sees to it
 
@@ -115,16 +139,19 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
       const int s = (k - k0) % NS;
       if (ok && !bar_wait(&empty[s], (uint32_t)((((k - k0) / NS) & 1) ^ 1))) { ok = false; report_error(err, 5); }
       if (ok && elect_one()) {
-        bar_expect(&full[s], L::STAGE);  // boxes are always complete: what lies outside the matrices is filled with zeros
+        bar_expect(&full[s], (uint32_t)(L::A_STAGE + bn * 128));  // boxes are always complete: what lies outside the matrices is filled with zeros
         asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
                      ::"r"(base + (uint32_t)(s * L::STAGE + L::A_STAGE)), "l"(&wmap), "r"(k * BK), "r"(z * a.rows + row0), "r"(s32(&full[s])) : "memory");
+        if constexpr (GLU)
+          asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
+                       ::"r"(base + (uint32_t)(s * L::STAGE + L::A_STAGE + width * 128)), "l"(&wmap), "r"(k * BK), "r"(a.rows + row0), "r"(s32(&full[s])) : "memory");
         asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
                      ::"r"(base + (uint32_t)(s * L::STAGE)), "l"(&xmap), "r"(z * a.xk + k * BK), "r"(tok0), "r"(s32(&full[s])) : "memory");
       }
       __syncwarp();
     }
   } else if (warp == W_MMA) {
-    constexpr uint32_t idesc = mma_desc<BN>();
+    const uint32_t idesc = mma_desc(bn);
     const uint32_t td = __shfl_sync(0xffffffffu, tmem, 0), base = __shfl_sync(0xffffffffu, s32(smem), 0);
     for (int k = k0; k < k1; ++k) {
       const int s = (k - k0) % NS;
@@ -149,7 +176,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
     if (!bar_wait(done, 0)) { ok = false; report_error(err, 5); }
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const int t = tok0 + 32 * warp + lane;
-    const int n_live = min(BN, a.rows - row0);
+    const int n_live = min(width, a.rows - row0);
     const int64_t off = (int64_t)t * a.y_ld + (int64_t)z * a.rows + row0;
     float* y = a.y ? a.y + slice * a.slice_stride + off : nullptr;
     __nv_bfloat16* y16 = a.y16 ? a.y16 + off : nullptr;
@@ -158,20 +185,18 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
     const bool vec = ((a.y_ld | a.rows) & 7) == 0;  // every run of eight results starts on a 16-byte boundary in either format
 #pragma unroll 1
     for (int c0 = 0; c0 < n_live; c0 += 32) {
-      uint32_t v[32];
-      asm volatile(
-          "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"
-          "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-          : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
-            "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]),
-            "=r"(v[16]), "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]),
-            "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-          : "r"(tmem + ((uint32_t)(32 * warp) << 16) + (uint32_t)c0) : "memory");
+      uint32_t v[32], u[32];
+      const uint32_t taddr = tmem + ((uint32_t)(32 * warp) << 16) + (uint32_t)c0;
+      load32(taddr, v);
+      if constexpr (GLU) load32(taddr + (uint32_t)width, u);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       if (t < a.tokens) {
         float f[32];
 #pragma unroll
-        for (int j = 0; j < 32; ++j) f[j] = a.gate ? __uint_as_float(v[j]) * gate : __uint_as_float(v[j]);
+        for (int j = 0; j < 32; ++j) {
+          if constexpr (GLU) f[j] = glu_of(__uint_as_float(v[j]), __uint_as_float(u[j]), a.glu);
+          else f[j] = a.gate ? __uint_as_float(v[j]) * gate : __uint_as_float(v[j]);
+        }
         if (vec) {
 #pragma unroll
           for (int j = 0; j < 32; j += 8)
@@ -217,29 +242,37 @@ bool encode_rows(CUtensorMap* map, const void* base, int64_t cols, int64_t rows,
              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int BN>
+template <int BN, bool GLU>
 cudaError_t launch_tiles(const Bf16Product& p, const Args& a, cudaStream_t stream, int* err) {
   CUtensorMap xmap, wmap;
-  if (!encode_rows(&xmap, p.x16, p.x_cols, p.tokens, p.x_ld, BM) || !encode_rows(&wmap, p.w, p.cols, (int64_t)p.rows * p.batch, p.cols, BN))
+  const int width = GLU ? a.bn / 2 : a.bn;  // rows of one box of W
+  if (!encode_rows(&xmap, p.x16, p.x_cols, p.tokens, p.x_ld, BM) || !encode_rows(&wmap, p.w, p.cols, (int64_t)p.rows * (GLU ? 2 : p.batch), p.cols, width))
     return cudaErrorInvalidValue;
   constexpr int smem = Lay<BN>::TOTAL;
   static PerDevice ready;
   std::atomic<int>& slot = ready.here();
   if (slot.load(std::memory_order_relaxed) == 0) {
-    const cudaError_t e = cudaFuncSetAttribute(gemm_bf16_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    const cudaError_t e = cudaFuncSetAttribute(gemm_bf16_kernel<BN, GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return e;
     slot.store(1, std::memory_order_relaxed);
   }
-  const dim3 grid((unsigned)((p.rows + BN - 1) / BN), (unsigned)((p.tokens + BM - 1) / BM), (unsigned)(p.batch * a.slices));
-  gemm_bf16_kernel<BN><<<grid, THREADS, smem, stream>>>(xmap, wmap, a, err);
+  const dim3 grid((unsigned)((p.rows + width - 1) / width), (unsigned)((p.tokens + BM - 1) / BM), (unsigned)(p.batch * a.slices));
+  gemm_bf16_kernel<BN, GLU><<<grid, THREADS, smem, stream>>>(xmap, wmap, a, err);
   return cudaGetLastError();
 }
 
+constexpr int SMS = 148;
 int tiles_of(int tokens, int rows, int batch, int bn) { return ((tokens + BM - 1) / BM) * ((rows + bn - 1) / bn) * batch; }
-int tile_width(int tokens, int rows, int batch) {
-  // the widest tile that still gives most SMs one
-  if (tiles_of(tokens, rows, batch, 256) >= 132) return 256;
-  return rows > 64 ? 128 : 64;
+// Width of a tile: with many tiles the one of 160 .. 256 (a multiple of `step`, so that both halves of a gated tile are
+// whole boxes of eight-row groups) whose waves over the SMs cost least; otherwise 128 or 64.
+int tile_width(int tokens, int rows, int batch, int step = 16) {
+  if (tiles_of(tokens, rows, batch, 256) < 132) return rows > 64 ? 128 : 64;
+  int best = 256, cost = 1 << 30;
+  for (int bn = 256; bn >= 160; bn -= step) {
+    const int c = ((tiles_of(tokens, rows, batch, bn) + SMS - 1) / SMS) * (bn + 24);  // 24: what a tile costs besides its columns
+    if (c < cost) { cost = c; best = bn; }
+  }
+  return best;
 }
 
 }  // namespace
@@ -252,7 +285,7 @@ bool gemm_bf16_supported(const void* w, int64_t rows, int64_t cols) {
 // least 512 columns long
 int gemm_bf16_slices(int tokens, int rows, int cols) {
   const int bn = tile_width(tokens, rows, 1);
-  if (bn == 256) return 1;
+  if (bn > 128) return 1;
   const int tiles = tiles_of(tokens, rows, 1, bn), nk = (cols + BK - 1) / BK;
   int s = 1;
   while (s < 8 && tiles * s * 2 <= 296 && nk / (s * 2) >= 8) s *= 2;
@@ -263,7 +296,8 @@ int gemm_bf16_slices(int tokens, int rows, int cols) {
 cudaError_t launch_gemm_bf16(const Bf16Product& p, cudaStream_t stream, int* err, uint64_t* launches) {
   if (p.tokens <= 0) return cudaSuccess;
   if (!gemm_bf16_supported(p.w, p.rows, p.cols) || p.batch < 1 || p.x_ld % 8 != 0 || (p.batch > 1 && p.xk % 8 != 0) || ((uintptr_t)p.x16 & 15) != 0 ||
-      (((uintptr_t)p.y | (uintptr_t)p.y16) & 15) != 0 || p.slices < 1 || (p.slices > 1 && (p.batch != 1 || p.y16 || p.gate)))
+      (((uintptr_t)p.y | (uintptr_t)p.y16) & 15) != 0 || p.slices < 1 || (p.slices > 1 && (p.batch != 1 || p.y16 || p.gate || p.glu)) ||
+      (p.glu && (p.batch != 1 || p.gate)))
     return cudaErrorInvalidValue;
   Args a{};
   a.y = p.y; a.y16 = (__nv_bfloat16*)p.y16; a.gate = p.gate;
@@ -272,11 +306,14 @@ cudaError_t launch_gemm_bf16(const Bf16Product& p, cudaStream_t stream, int* err
   a.batch = p.batch; a.slices = p.slices;
   if ((a.slices - 1) * ((a.nk + a.slices - 1) / a.slices) >= a.nk) return cudaErrorInvalidValue;
   if (launches) ++*launches;
-  switch (tile_width(p.tokens, p.rows, p.batch)) {
-    case 256: return launch_tiles<256>(p, a, stream, err);
-    case 128: return launch_tiles<128>(p, a, stream, err);
-    default: return launch_tiles<64>(p, a, stream, err);
+  if (p.glu) {
+    a.glu = *p.glu;
+    a.bn = std::max(tile_width(p.tokens, 2 * p.rows, 1, 32), 128);
+    return a.bn > 128 ? launch_tiles<256, true>(p, a, stream, err) : launch_tiles<128, true>(p, a, stream, err);
   }
+  a.bn = tile_width(p.tokens, p.rows, p.batch);
+  if (a.bn > 128) return launch_tiles<256, false>(p, a, stream, err);
+  return a.bn == 128 ? launch_tiles<128, false>(p, a, stream, err) : launch_tiles<64, false>(p, a, stream, err);
 }
 
 }  // namespace llr

@@ -9,6 +9,8 @@
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
 
+#include <algorithm>
+
 #include "llr_formats.cuh"
 #include "llr_kernels.cuh"
 
@@ -105,6 +107,75 @@ gemv_rows_kernel(const uint8_t* __restrict__ W, int64_t row_bytes, int64_t rows,
   }
 }
 
+// Rows i and n + i of a stacked gate | up matrix by one warp, which then has both factors of result i: half the pieces in
+// flight per row, two rows at a time.
+template <int DT, int MT>
+__global__ void __launch_bounds__(ROW_WARPS * 32, (DT == DT_F32 || MT > 2) ? 2 : 4)
+gemv_rows_glu_kernel(const uint8_t* __restrict__ W, int64_t row_bytes, int64_t cols, const float* __restrict__ X, float* __restrict__ Y, int tokens,
+                     GluShape glu) {
+  const int lane = threadIdx.x & 31;
+  const int64_t warp = (int64_t)blockIdx.x * ROW_WARPS + (threadIdx.x >> 5), n_warps = (int64_t)gridDim.x * ROW_WARPS;
+  constexpr int UNROLL = Unroll<DT>::N / 2;
+  for (int64_t row = warp; row < glu.n; row += n_warps) {
+    const uint8_t* wr[2] = {W + row * row_bytes, W + (row + glu.n) * row_bytes};
+    float acc[2][MT];
+#pragma unroll
+    for (int t = 0; t < MT; ++t) acc[0][t] = acc[1][t] = 0.f;
+    for (int64_t c0 = 8 * lane; c0 < cols; c0 += 256 * UNROLL) {
+      Raw8<DT> raw[2][UNROLL];
+#pragma unroll
+      for (int i = 0; i < UNROLL; ++i)
+        if (c0 + 256 * i < cols) { fetch8<DT>(wr[0], c0 + 256 * i, raw[0][i]); fetch8<DT>(wr[1], c0 + 256 * i, raw[1][i]); }
+#pragma unroll
+      for (int i = 0; i < UNROLL; ++i) {
+        const int64_t c = c0 + 256 * i;
+        if (c < cols) {
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            float w[8];
+            widen8<DT>(raw[r][i], w);
+#pragma unroll
+            for (int t = 0; t < MT; ++t)
+              if (t < tokens) {
+                const float4* xp = (const float4*)(X + (int64_t)t * cols + c);
+                const float4 a = __ldg(xp), b = __ldg(xp + 1);
+                float s = acc[r][t];
+                s = fmaf(w[0], a.x, s); s = fmaf(w[1], a.y, s); s = fmaf(w[2], a.z, s); s = fmaf(w[3], a.w, s);
+                s = fmaf(w[4], b.x, s); s = fmaf(w[5], b.y, s); s = fmaf(w[6], b.z, s); s = fmaf(w[7], b.w, s);
+                acc[r][t] = s;
+              }
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < MT; ++t) {
+      float a = acc[0][t], b = acc[1][t];
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) { a += __shfl_xor_sync(~0u, a, o); b += __shfl_xor_sync(~0u, b, o); }
+      if (lane == 0 && t < tokens) {
+        a = fminf(a, glu.limit);
+        b = fminf(fmaxf(b, -glu.limit), glu.limit);
+        Y[(int64_t)t * glu.n + row] = __fmul_rn(__fmul_rn(a, __fdiv_rn(1.0f, 1.0f + expf(-__fmul_rn(glu.alpha, a)))), __fadd_rn(b, glu.shift));
+      }
+    }
+  }
+}
+
+template <int DT, int MT>
+cudaError_t launch_rows_glu(const MatView& m, const float* x, float* y, int tokens, const GluShape& glu, cudaStream_t stream, int sm_count) {
+  const int64_t grid = std::min<int64_t>((glu.n + ROW_WARPS - 1) / ROW_WARPS, (int64_t)sm_count * 8);
+  gemv_rows_glu_kernel<DT, MT><<<(unsigned)grid, ROW_WARPS * 32, 0, stream>>>(m.w, m.row_bytes, m.cols, x, y, tokens, glu);
+  return cudaGetLastError();
+}
+template <int DT>
+cudaError_t launch_rows_glu_mt(const MatView& m, const float* x, float* y, int tokens, const GluShape& glu, cudaStream_t stream, int sm_count) {
+  if (tokens == 1) return launch_rows_glu<DT, 1>(m, x, y, tokens, glu, stream, sm_count);
+  if (tokens == 2) return launch_rows_glu<DT, 2>(m, x, y, tokens, glu, stream, sm_count);
+  if (tokens <= 4) return launch_rows_glu<DT, 4>(m, x, y, tokens, glu, stream, sm_count);
+  return launch_rows_glu<DT, 8>(m, x, y, tokens, glu, stream, sm_count);
+}
+
 template <int DT, int MT>
 cudaError_t launch_rows(const MatView& m, const float* x, float* y, int tokens, cudaStream_t stream, int sm_count) {
   int64_t grid = (m.rows + ROW_WARPS - 1) / ROW_WARPS;
@@ -123,6 +194,15 @@ cudaError_t launch_rows_mt(const MatView& m, const float* x, float* y, int token
 }
 
 }  // namespace
+
+cudaError_t launch_gemv_rows_glu(const MatView& m, const float* x, float* out, const GluShape& glu, int tokens, cudaStream_t stream, int sm_count,
+                                 uint64_t* launches) {
+  if (!gemv_rows_supported(m) || m.rows != 2 * (int64_t)glu.n || tokens < 1 || tokens > 8 || ((uintptr_t)x & 15) != 0) return cudaErrorInvalidValue;
+  if (launches) ++*launches;
+  if (m.dtype == DT_F32) return launch_rows_glu_mt<DT_F32>(m, x, out, tokens, glu, stream, sm_count);
+  if (m.dtype == DT_F16) return launch_rows_glu_mt<DT_F16>(m, x, out, tokens, glu, stream, sm_count);
+  return launch_rows_glu_mt<DT_BF16>(m, x, out, tokens, glu, stream, sm_count);
+}
 
 bool gemv_rows_supported(const MatView& m) {
   if (m.dtype != DT_F32 && m.dtype != DT_F16 && m.dtype != DT_BF16) return false;

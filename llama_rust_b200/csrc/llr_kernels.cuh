@@ -66,6 +66,11 @@ bool gemv_rows_supported(const MatView& m);
 cudaError_t launch_gemv_rows(const MatView& m, const float* x, float* y, int64_t tokens, cudaStream_t stream, int sm_count,
                              uint64_t* launches);
 
+struct GluShape;
+// A stacked gate | up matrix (2 n rows) and the clamped gated unit of its products in one launch (tokens <= 8): out[t][i]
+cudaError_t launch_gemv_rows_glu(const MatView& m, const float* x, float* out, const GluShape& glu, int tokens, cudaStream_t stream,
+                                 int sm_count, uint64_t* launches);
+
 // Integer tensor-core decode GEMV for Q4_K / Q6_K / Q8_0 (tokens <= 8 per pass); see
 // llr_gemv_stream.cu.  Launched with programmatic stream serialization.
 bool gemv_mma_supported(const MatView& m);
@@ -300,6 +305,8 @@ cudaError_t launch_argmax_advance(const float* logits, int n, int* out_id, float
 cudaError_t launch_argmax_rows(const float* logits, int n_rows, int n, int* out_id, float* out_margin, cudaStream_t s,
                                uint64_t* launches);
 
+// Clamped gated unit: a * sigmoid(alpha * a) * (b + shift), a = min(gate, limit), b = clamp(up, -limit, limit); n results
+struct GluShape { int n; float limit, alpha, shift; };
 // ---- products with bfloat16 weights for many rows (llr_gemm_bf16.cu): tcgen05, bfloat16 activations, f32 accumulation ----
 // y[t * y_ld + z * rows + r] = sum_c W[z * rows + r][c] x[t][z * xk + c] for z < batch (a product per head), times
 // sigmoid(gate[t * gate_ld + z]) when gate is set.  Results as f32 (y), as bfloat16 (y16), or both.  With slices > 1
@@ -313,6 +320,7 @@ struct Bf16Product {
   const float* gate;
   int64_t y_ld, gate_ld, slice_stride;
   int tokens, rows, cols, batch, xk, slices;
+  const GluShape* glu;  // W stacks gate | up, 2 rows rows: the results are clamped gated units (batch 1)
 };
 bool gemm_bf16_supported(const void* w, int64_t rows, int64_t cols);
 int gemm_bf16_slices(int tokens, int rows, int cols);
@@ -364,16 +372,22 @@ cudaError_t launch_head_transpose(const void* w, int heads, int rows, int cols, 
 // Attention over the visible keys.  q: row t at q + t * q_ld.  Result rows of n_head * dv, f32 (out) and/or bfloat16 (out16);
 // gate (may be null): element gate, result times sigmoid(gate[t * gate_ld + h * dv + i]).
 // one_sequence: the rows are one sequence at consecutive positions; with tensor_cores such rows may run as binary16 MMAs.
-size_t span_scratch_floats(const SpanShape& sh);
+// A single decode token whose projection the attention kernel takes in itself (null proj: it is in the cache already):
+// the row's stacked q | k | v with launch_qkv_store's arguments, or (latent) its latent with the weights in k_norm.
+struct NewToken {
+  const float *proj = nullptr, *bias = nullptr, *q_norm = nullptr, *k_norm = nullptr;
+  float eps = 0.f;
+  bool latent = false;
+};
+size_t span_scratch_floats(const SpanShape& sh, int max_rows);
 bool span_supported(const SpanShape& sh);
 cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape& sh, const LayerKv& kv, const RowMap& rows, int t0, int tokens,
                                   float* out, void* out16, const float* gate, int64_t gate_ld, float* scratch, bool tensor_cores,
-                                  bool one_sequence, cudaStream_t s, uint64_t* launches);
+                                  bool one_sequence, const NewToken* nt, cudaStream_t s, uint64_t* launches);
 // x[t] += y[t] / rms(y[t]) * w, y given as `slices` partial sums `slice_stride` floats apart; x16 (may be null): the new x
 cudaError_t launch_norm_add(float* x, const float* y, int slices, int64_t slice_stride, const float* w, float eps, void* x16, int tokens, int n,
                             cudaStream_t s, uint64_t* launches);
-// out[t][i] = a * sigmoid(alpha * a) * (b + shift), a = min(gu[t][i], limit), b = clamp(gu[t][n + i], -limit, limit)
-struct GluShape { int n; float limit, alpha, shift; };
+// the clamped gated unit of a stacked product: row t of gu is gate | up, n each
 cudaError_t launch_clamped_glu(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches);
 
 // *flag_dev = 1 when the two device byte ranges differ (both 16-byte aligned), else 0

@@ -132,7 +132,7 @@ cudaError_t layered_layers(llr_session* s, const int* ids_dev, size_t n, const R
     const float* q = D.proj;
     int64_t q_ld = L.in_rows;
     if (latent) {
-      if (L.own_kv && (ce = launch_latent_store(D.proj + L.q_rows, L.in_rows, L.kv_norm, (int)mx.kv_rank, D.eps, kv, rows, N, st, lc)) != cudaSuccess) return ce;
+      if (n > 1 && L.own_kv && (ce = launch_latent_store(D.proj + L.q_rows, L.in_rows, L.kv_norm, (int)mx.kv_rank, D.eps, kv, rows, N, st, lc)) != cudaSuccess) return ce;
       // queries into the latent space, head by head
       if (up_tc) {
         if ((ce = launch_rows_bf16(D.proj, L.in_rows, L.q_rows, D.a16, N, st, lc)) != cudaSuccess) return ce;
@@ -146,7 +146,7 @@ cudaError_t layered_layers(llr_session* s, const int* ids_dev, size_t n, const R
       if (ce != cudaSuccess) return ce;
       q = D.lat_q;
       q_ld = (int64_t)mx.n_head * mx.kv_rank;
-    } else {
+    } else if (n > 1) {
       const QkvShape sh{(int)mx.n_head, (int)mx.n_head_kv, (int)mx.dim, (int)mx.vdim, D.eps};
       if ((ce = launch_qkv_store(D.proj, L.in_rows, L.in_bias, L.q_norm, L.k_norm, sh, kv, rows, N, st, lc)) != cudaSuccess) return ce;
     }
@@ -155,9 +155,16 @@ cudaError_t layered_layers(llr_session* s, const int* ids_dev, size_t n, const R
     float* o = o16 ? nullptr : latent ? D.lat_o : D.att;
     void* ob = o16 ? D.a16 : nullptr;
     const float* egate = latent ? nullptr : gate;
+    NewToken nt;  // a single token: the attention kernel norms and stores it
+    nt.eps = D.eps;
+    nt.latent = latent;
+    if (n == 1 && L.own_kv) nt.proj = latent ? D.proj + L.q_rows : D.proj;
+    nt.bias = L.in_bias;
+    nt.q_norm = L.q_norm;
+    nt.k_norm = latent ? L.kv_norm : L.k_norm;
     auto attend = [&](size_t t0, size_t len, bool one) {
       return launch_span_attention(q, q_ld, L.span, kv, rows, (int)t0, (int)len, o, ob, egate, L.in_rows, D.scratch, tc && len >= (size_t)BF16_TC_MIN_TOKENS, one,
-                                   st, lc);
+                                   &nt, st, lc);
     };
     if (!rows.row_seq) {
       ce = attend(0, n, true);
@@ -198,8 +205,18 @@ cudaError_t layered_layers(llr_session* s, const int* ids_dev, size_t n, const R
     if (L.mlp.n_ff == 0) continue;
     const GluShape glu{(int)L.mlp.n_ff, L.mlp.limit, L.mlp.alpha, L.mlp.shift};
     const bool down_tc = tc && L.tc_down;
-    if ((ce = product(L.mlp.gate_up, tc && L.tc_gu, s->x, D.x16, D.gu, nullptr)) != cudaSuccess ||
-        (ce = launch_clamped_glu(D.gu, glu, down_tc ? nullptr : D.act, down_tc ? D.a16 : nullptr, N, st, lc)) != cudaSuccess ||
+    const MatView gu = view_of(L.mlp.gate_up);
+    if (tc && L.tc_gu) {  // the gated unit in the product's epilogue
+      Bf16Product p{};
+      p.w = gu.w; p.x16 = D.x16; p.x_ld = p.x_cols = E; p.y = down_tc ? nullptr : D.act; p.y16 = down_tc ? D.a16 : nullptr; p.y_ld = glu.n;
+      p.tokens = N; p.rows = glu.n; p.cols = E; p.batch = 1; p.slices = 1; p.glu = &glu;
+      ce = launch_gemm_bf16(p, st, e->err_flag, lc);
+    } else if (e->path == PATH_AUTO && n <= 8 && !down_tc && gemv_rows_supported(gu)) {
+      ce = launch_gemv_rows_glu(gu, s->x, D.act, glu, N, st, e->sm_count, lc);
+    } else if ((ce = product(L.mlp.gate_up, false, s->x, nullptr, D.gu, nullptr)) == cudaSuccess) {
+      ce = launch_clamped_glu(D.gu, glu, down_tc ? nullptr : D.act, down_tc ? D.a16 : nullptr, N, st, lc);
+    }
+    if (ce != cudaSuccess ||
         (ce = product(L.mlp.down, down_tc, D.act, D.a16, D.y, &slices)) != cudaSuccess ||
         (ce = launch_norm_add(s->x, D.y, slices, (int64_t)n * E, L.mlp_norm, D.eps, tc ? D.x16 : nullptr, N, E, st, lc)) != cudaSuccess)
       return ce;
@@ -266,7 +283,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
       b16 = std::max(b16, H * x.vdim);
     }
     ff = std::max(ff, (size_t)L.mlp.n_ff);
-    scratch = std::max(scratch, span_scratch_floats(L.span));
+    scratch = std::max(scratch, span_scratch_floats(L.span, 512));
   }
   a16 = std::max(a16, ff);
   llr_session* s = new (std::nothrow) llr_session();

@@ -27,6 +27,10 @@ __device__ __forceinline__ uint2 pack4_bf16(float4 v) {
   return make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
 }
 
+__device__ __forceinline__ float4 widen4(uint2 u) {
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+}
+
 // ---- embedding ------------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256)
 embed_kernel(const uint16_t* __restrict__ table, const uint16_t* __restrict__ pos_table, const int* __restrict__ ids, RowMap rows, float scale,
@@ -35,11 +39,15 @@ embed_kernel(const uint16_t* __restrict__ table, const uint16_t* __restrict__ po
   const int t = blockIdx.x;
   const uint16_t* e = table + (int64_t)ids[t] * n;
   const uint16_t* p = pos_table ? pos_table + (int64_t)row_position(rows, t) * n : nullptr;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    float v = __fmul_rn(bf(e[i]), scale);
-    if (p) v = __fadd_rn(v, bf(p[i]));
-    x[(int64_t)t * n + i] = v;
-    if (x16) x16[(int64_t)t * n + i] = __float2bfloat16_rn(v);
+  for (int i = 4 * threadIdx.x; i < n; i += 4 * blockDim.x) {  // n is a multiple of four
+    float4 v = widen4(*(const uint2*)(e + i));
+    v = make_float4(__fmul_rn(v.x, scale), __fmul_rn(v.y, scale), __fmul_rn(v.z, scale), __fmul_rn(v.w, scale));
+    if (p) {
+      const float4 u = widen4(*(const uint2*)(p + i));
+      v = make_float4(__fadd_rn(v.x, u.x), __fadd_rn(v.y, u.y), __fadd_rn(v.z, u.z), __fadd_rn(v.w, u.w));
+    }
+    *(float4*)(x + (int64_t)t * n + i) = v;
+    if (x16) *(uint2*)(x16 + (int64_t)t * n + i) = pack4_bf16(v);
   }
 }
 
@@ -52,56 +60,98 @@ __device__ __forceinline__ float inv_rms(float sum_sq, int n, float eps) {
   return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(sum_sq, (float)n), eps)));
 }
 
+// A row of the stacked q | k | v projection: biases, and the factors that norm all of q and all of k.  Blocks of
+// PROJ_THREADS threads; each sum is formed in one order whichever kernel asks for it.
+constexpr int PROJ_THREADS = 256;
+struct QkvRow {
+  const float *p, *bias, *q_norm, *k_norm;
+  float qi, ki;
+  int nq, nk;
+  __device__ __forceinline__ float q(int i) const {
+    const float v = bias ? __fadd_rn(p[i], bias[i]) : p[i];
+    return q_norm ? __fmul_rn(__fmul_rn(v, qi), q_norm[i]) : v;
+  }
+  __device__ __forceinline__ float k(int i) const {
+    const float v = bias ? __fadd_rn(p[nq + i], bias[nq + i]) : p[nq + i];
+    return k_norm ? __fmul_rn(__fmul_rn(v, ki), k_norm[i]) : v;
+  }
+  __device__ __forceinline__ float v(int i) const { return bias ? __fadd_rn(p[nq + nk + i], bias[nq + nk + i]) : p[nq + nk + i]; }
+};
+// a thread's share of the sum of (p + bias)^2; p and bias are 16-byte aligned and n is a multiple of four when vec
+__device__ __forceinline__ float sum_squares(const float* p, const float* bias, int n, bool vec) {
+  float s = 0.f;
+  if (vec) {
+#pragma unroll 4
+    for (int i = 4 * threadIdx.x; i < n; i += 4 * PROJ_THREADS) {
+      float4 v = *(const float4*)(p + i);
+      if (bias) {
+        const float4 u = *(const float4*)(bias + i);
+        v = make_float4(__fadd_rn(v.x, u.x), __fadd_rn(v.y, u.y), __fadd_rn(v.z, u.z), __fadd_rn(v.w, u.w));
+      }
+      s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += PROJ_THREADS) {
+      const float v = bias ? __fadd_rn(p[i], bias[i]) : p[i];
+      s = fmaf(v, v, s);
+    }
+  }
+  return s;
+}
+__device__ __forceinline__ QkvRow qkv_row(const float* p, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh,
+                                          float (*red)[32]) {
+  const int nq = sh.n_head * sh.dk, nk = sh.n_kv * sh.dk;
+  const bool vec = ((ld | nq | nk) & 3) == 0;
+  QkvRow r{p, bias, q_norm, k_norm, 1.f, 1.f, nq, nk};
+  const float qs = q_norm ? sum_squares(p, bias, nq, vec) : 0.f, ks = k_norm ? sum_squares(p + nq, bias ? bias + nq : nullptr, nk, vec) : 0.f;
+  if (q_norm) r.qi = inv_rms(block_sum(qs, red[0]), nq, sh.eps);
+  if (k_norm) r.ki = inv_rms(block_sum(ks, red[1]), nk, sh.eps);
+  return r;
+}
+
 // one block per row
-__global__ void __launch_bounds__(512)
-qkv_store_kernel(float* __restrict__ proj, int ld, const float* __restrict__ bias, const float* __restrict__ q_norm,
+__global__ void __launch_bounds__(PROJ_THREADS)
+qkv_store_kernel(float* proj, int ld, const float* __restrict__ bias, const float* __restrict__ q_norm,
                  const float* __restrict__ k_norm, QkvShape sh, LayerKv kv, RowMap rows) {
   pdl_enter();
-  __shared__ float s1[32], s2[32];
-  const int t = blockIdx.x, nq = sh.n_head * sh.dk, nk = sh.n_kv * sh.dk, nv = sh.n_kv * sh.dv;
+  __shared__ float red[2][32];
+  const int t = blockIdx.x, nk = sh.n_kv * sh.dk, nv = sh.n_kv * sh.dv;
   float* p = proj + (int64_t)t * ld;
-  float qs = 0.f, ks = 0.f;
-  if (bias || q_norm || k_norm) {
-    for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
-      float v = p[i];
-      if (bias) { v = __fadd_rn(v, bias[i]); p[i] = v; }  // read back below by the same thread
-      if (i < nq) qs = fmaf(v, v, qs); else ks = fmaf(v, v, ks);
-    }
-    qs = block_sum(qs, s1);
-    ks = block_sum(ks, s2);
-  }
+  const QkvRow r = qkv_row(p, ld, bias, q_norm, k_norm, sh, red);
   const int pos = row_position(rows, t), seq = row_sequence(rows, t);
-  const float qi = q_norm ? inv_rms(qs, nq, sh.eps) : 1.f, ki = k_norm ? inv_rms(ks, nk, sh.eps) : 1.f;
-  for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
-    const float v = p[i];
-    if (i < nq) {
-      if (q_norm) p[i] = __fmul_rn(__fmul_rn(v, qi), q_norm[i]);
-    } else {
-      const int c = i - nq;
-      kv.k[slot_of(kv, seq, pos, kv.k_block, c / sh.dk, sh.dk) + c % sh.dk] = k_norm ? __fmul_rn(__fmul_rn(v, ki), k_norm[c]) : v;
+  // the page and the place in it once; heads lie block_tokens vectors apart
+  float* k0 = kv.k + slot_of(kv, seq, pos, kv.k_block, 0, sh.dk);
+  float* v0 = kv.v + slot_of(kv, seq, pos, kv.v_block, 0, sh.dv);
+  for (int i = threadIdx.x; i < nk; i += PROJ_THREADS) k0[(int64_t)(i / sh.dk) * kv.block_tokens * sh.dk + i % sh.dk] = r.k(i);
+  for (int i = threadIdx.x; i < nv; i += PROJ_THREADS) v0[(int64_t)(i / sh.dv) * kv.block_tokens * sh.dv + i % sh.dv] = r.v(i);
+  if (bias || q_norm) {
+    for (int i0 = threadIdx.x; i0 < r.nq; i0 += 4 * PROJ_THREADS) {  // four values in flight; each is read and written by one thread
+      float u[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) u[j] = i0 + j * PROJ_THREADS < r.nq ? r.q(i0 + j * PROJ_THREADS) : 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (i0 + j * PROJ_THREADS < r.nq) p[i0 + j * PROJ_THREADS] = u[j];
     }
-  }
-  for (int c = threadIdx.x; c < nv; c += blockDim.x) {
-    float v = p[nq + nk + c];
-    if (bias) v = __fadd_rn(v, bias[nq + nk + c]);
-    kv.v[slot_of(kv, seq, pos, kv.v_block, c / sh.dv, sh.dv) + c % sh.dv] = v;
   }
 }
 
-__global__ void __launch_bounds__(256)
-latent_store_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w, int n, float eps, LayerKv kv, RowMap rows) {
-  pdl_enter();
-  __shared__ float sh[32];
-  const int t = blockIdx.x;
-  const float* p = proj + (int64_t)t * ld;
+// the latent of a row: normed, weighted, into the cache
+__device__ __forceinline__ void store_latent(const float* p, const float* w, int n, float eps, float* c, float* red) {
   float ss = 0.f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(p[i], p[i], ss);
-  const float inv = inv_rms(block_sum(ss, sh), n, eps);
-  float* c = kv.k + slot_of(kv, row_sequence(rows, t), row_position(rows, t), kv.k_block, 0, n);
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+  for (int i = threadIdx.x; i < n; i += PROJ_THREADS) ss = fmaf(p[i], p[i], ss);
+  const float inv = inv_rms(block_sum(ss, red), n, eps);
+  for (int i = threadIdx.x; i < n; i += PROJ_THREADS) {
     const float v = __fmul_rn(p[i], inv);
     c[i] = w ? __fmul_rn(v, w[i]) : v;
   }
+}
+__global__ void __launch_bounds__(PROJ_THREADS)
+latent_store_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ w, int n, float eps, LayerKv kv, RowMap rows) {
+  pdl_enter();
+  __shared__ float red[32];
+  const int t = blockIdx.x;
+  store_latent(proj + (int64_t)t * ld, w, n, eps, kv.k + slot_of(kv, row_sequence(rows, t), row_position(rows, t), kv.k_block, 0, n), red);
 }
 
 __global__ void __launch_bounds__(256)
@@ -239,10 +289,16 @@ struct KvSpan {
 };
 
 // grid (kv head x group of at most ATT_MAX_GQA query heads, slice of the visible keys, row)
+// With nt (a single decode token) the kernel also does what the store kernels do for that token: the query is biased and
+// normed as it is loaded, and the blocks whose slice holds the token's own position write its key and value (or its
+// latent) into the cache and read them back like any other; blocks that share a kv head write the same values.
+static_assert(PROJ_THREADS == ATT_THREADS, "the sums over a projection are formed in one order");
 template <int MAX_VALUE>
 __global__ void __launch_bounds__(ATT_THREADS)
-span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv kv, RowMap rows, int t0, int chunk, float* __restrict__ part) {
+span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv kv, RowMap rows, int t0, int chunk, float* __restrict__ part,
+                    NewToken nt) {
   pdl_enter();
+  __shared__ float red[2][32];
   extern __shared__ float sm[];  // q [heads][dk] | scores [heads][chunk] or sums [P][heads][dv]
   const int gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
   const int head = blockIdx.x / groups, g0 = (blockIdx.x % groups) * ATT_MAX_GQA, heads = min(ATT_MAX_GQA, gq - g0);
@@ -253,14 +309,27 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
   if (s0 >= span.n) return;
   float* sq = sm;
   float* sc = sq + heads * sh.dk;
-  for (int i = threadIdx.x; i < heads * sh.dk; i += ATT_THREADS) sq[i] = q[(int64_t)t * q_ld + (int64_t)h0 * sh.dk + i];
+  if (nt.proj && !nt.latent) {
+    const QkvShape qs{sh.n_head, sh.n_kv, sh.dk, sh.dv, nt.eps};
+    const QkvRow r = qkv_row(nt.proj, (int)q_ld, nt.bias, nt.q_norm, nt.k_norm, qs, red);
+    for (int i = threadIdx.x; i < heads * sh.dk; i += ATT_THREADS) sq[i] = r.q(h0 * sh.dk + i);
+    if (s1 == span.n) {
+      float* k = kv.k + slot_of(kv, row_sequence(rows, t), pos, kv.k_block, head, sh.dk);
+      float* v = kv.v + slot_of(kv, row_sequence(rows, t), pos, kv.v_block, head, sh.dv);
+      for (int i = threadIdx.x; i < sh.dk; i += ATT_THREADS) k[i] = r.k(head * sh.dk + i);
+      for (int i = threadIdx.x; i < sh.dv; i += ATT_THREADS) v[i] = r.v(head * sh.dv + i);
+    }
+  } else {
+    for (int i = threadIdx.x; i < heads * sh.dk; i += ATT_THREADS) sq[i] = q[(int64_t)t * q_ld + (int64_t)h0 * sh.dk + i];
+    if (nt.proj && s1 == span.n) store_latent(nt.proj, nt.k_norm, sh.dk, nt.eps, kv.k + slot_of(kv, row_sequence(rows, t), pos, kv.k_block, 0, sh.dk), red[0]);
+  }
   __syncthreads();
   // records: [row of the pass][query head][slice][dv + 2]; a group's heads follow each other n_split records apart
   float* rec = part + (((int64_t)blockIdx.z * sh.n_kv * groups + blockIdx.x) * n_split + split) * ATT_MAX_GQA * (sh.dv + 2);
   attend_slice<MAX_VALUE>(KvSpan{kv, sh, span, row_sequence(rows, t), head, pos, h0}, sq, sc, rec, s0, s1, chunk, sh.dk, sh.dv, heads);
 }
 
-// grid (query head, row): merges a head's slices (at most 32) and applies the element gate
+// grid (query head, row, 128 dimensions): merges a head's slices (at most 32) and applies the element gate
 __global__ void __launch_bounds__(128)
 span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, int t0, int chunk, int n_split, float* __restrict__ out,
                     __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate, int64_t gate_ld) {
@@ -275,34 +344,37 @@ span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, i
   const float m = warp_max(ms);
   const float e = lane < used ? expf(ms - m) : 0.f;
   const float l = warp_sum(lane < used ? base[lane * stride + sh.dv + 1] * e : 0.f);
-  for (int i0 = 0; i0 < sh.dv; i0 += 128) {
-    const int i = i0 + threadIdx.x;
-    const bool live = i < sh.dv;
-    float acc = 0.f;
-    for (int sp = 0; sp < used; sp += 4) {
-      float v[4];
+  const int i = blockIdx.z * 128 + threadIdx.x;
+  const bool live = i < sh.dv;
+  float acc = 0.f;
+  for (int sp = 0; sp < used; sp += 8) {  // eight slices' values are fetched before the first is used
+    float v[8];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) v[j] = (live && sp + j < used) ? base[(sp + j) * stride + i] : 0.f;
+    for (int j = 0; j < 8; ++j) v[j] = (live && sp + j < used) ? base[(sp + j) * stride + i] : 0.f;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc = fmaf(v[j], __shfl_sync(~0u, e, (sp + j) & 31), acc);  // a slice beyond `used` has value 0 and weight 0
-    }
-    if (live) {
-      float r = __fdiv_rn(acc, l);
-      const int64_t o = (int64_t)h * sh.dv + i;
-      if (gate) r = __fmul_rn(r, sigmoid(gate[(int64_t)t * gate_ld + o]));
-      if (out) out[(int64_t)t * sh.n_head * sh.dv + o] = r;
-      if (out16) out16[(int64_t)t * sh.n_head * sh.dv + o] = __float2bfloat16_rn(r);
-    }
+    for (int j = 0; j < 8; ++j) acc = fmaf(v[j], __shfl_sync(~0u, e, (sp + j) & 31), acc);  // a slice beyond `used` has value 0 and weight 0
+  }
+  if (live) {
+    float r = __fdiv_rn(acc, l);
+    const int64_t o = (int64_t)h * sh.dv + i;
+    if (gate) r = __fmul_rn(r, sigmoid(gate[(int64_t)t * gate_ld + o]));
+    if (out) out[(int64_t)t * sh.n_head * sh.dv + o] = r;
+    if (out16) out16[(int64_t)t * sh.n_head * sh.dv + o] = __float2bfloat16_rn(r);
   }
 }
 
 // ---- prompt chunks on the tensor cores ------------------------------------------------------------------------------
-// Rows of ONE sequence at consecutive positions.  A block takes one kv head and 64 (row, query head) pairs in row-major
-// order -- all query heads of a kv head share its keys, so any ratio of heads fills the tile (one latent for every head
-// included) -- and walks the keys that any of its rows sees, 64 at a time.  Queries (rescaled per pair by a power of two),
-// keys, values and the exponentials are rounded to binary16 operands; scores and sums are m16n8k16 MMAs with f32
-// accumulators; scale, distance bias, mask, maxima, exponentials and their sums are f32.
+// Rows of ONE sequence at consecutive positions.  The keys and values that any of the rows sees are first gathered from
+// their pages into contiguous binary16 rows (span_gather_kernel), so that the attention kernel copies tiles with 16-byte
+// asynchronous copies and neither looks pages up nor converts.
+// A block takes one kv head and 64 (row, query head) pairs in row-major order -- all query heads of a kv head share its
+// keys, so any ratio of heads fills the tile (one latent for every head included) -- and walks the keys that any of its
+// rows sees, 64 at a time.  Queries (rescaled per pair by a power of two), keys, values and the exponentials are
+// binary16 operands; scores and sums are m16n8k16 MMAs with f32 accumulators; scale, distance bias, mask, maxima,
+// exponentials and their sums are f32.
 // Sixteen pairs belong to NS warps: each scores 64 / NS of the keys and owns 8 ND of the value dimensions.
+// The copies run one tile ahead of their use: values arrive while their keys are scored, the next keys while the values
+// are added up; where keys and values are one latent there are two buffers instead.
 constexpr int CH = 64;
 __device__ __forceinline__ uint32_t pack_h2(float lo, float hi) {
   const __half2 h = __floats2half2_rn(lo, hi);
@@ -322,60 +394,101 @@ __device__ __forceinline__ void ldm4_t(uint32_t (&r)[4], const __half* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
 }
+__device__ __forceinline__ void copy16(const __half* dst, const __half* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void copy_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-struct MmaLayout {  // halves; widths are multiples of 16, so a pitch is an odd number of 16-byte units
-  int kw, vw, qp, kp, vp;
-  bool shared;  // values are the keys
+// Widths of the gathered rows and of the tiles, in halves; multiples of 16, so that a tile's pitch (width + 8) is an odd
+// number of 16-byte units.  Where values are the keys there is one row of the wider of the two.
+struct MmaLayout {
+  int kw, vw, kr, vr;  // score columns, value columns, gathered key row, gathered value row (0: the keys)
+  bool shared;
+  int qp, kp, vp;
 };
 inline __host__ __device__ MmaLayout mma_layout(int dk, int dv, int nd, int ns, bool shared) {
   MmaLayout L;
   L.kw = (dk + 15) / 16 * 16;
   L.vw = 8 * nd * ns;
   L.shared = shared;
+  L.kr = shared && L.vw > L.kw ? L.vw : L.kw;
+  L.vr = shared ? 0 : L.vw;
   L.qp = L.kw + 8;
-  L.kp = (shared && L.vw > L.kw ? L.vw : L.kw) + 8;
+  L.kp = L.kr + 8;
   L.vp = shared ? L.kp : L.vw + 8;
   return L;
 }
 inline __host__ __device__ size_t mma_smem(const MmaLayout& L, int ns) {
-  return ((size_t)64 * L.qp + (size_t)CH * L.kp + (L.shared ? 0 : (size_t)CH * L.vp) + (ns > 1 ? 64 * (CH + 8) : 0)) * 2;
+  return ((size_t)64 * L.qp + (size_t)CH * L.kp * (L.shared ? 2 : 1) + (L.shared ? 0 : (size_t)CH * L.vp) + (ns > 1 ? 64 * (CH + 8) : 0)) * 2;
+}
+
+// The list of keys a group of rows sees: kept tokens before the first row's window, then every position from there to the
+// last row.  Row m of the gathered keys of kv head g starts at k16 + ((int64_t)g * n + m) * kr.
+struct GroupKeys {
+  int lo, nk, n;
+  __device__ __forceinline__ int at(int m) const { return m < nk ? m : lo + m - nk; }
+  __device__ __forceinline__ int index(int j) const { return j < nk ? j : j - lo + nk; }  // of a position in the list
+};
+__device__ __forceinline__ GroupKeys group_keys(int first, int rows, int window, int keep_first) {
+  const int lo = window > 0 ? max(0, first - window + 1) : 0, nk = min(keep_first, lo);
+  return GroupKeys{lo, nk, nk + first + rows - lo};
+}
+
+// one warp per key row: grid (keys / 8, kv head)
+__global__ void __launch_bounds__(256)
+span_gather_kernel(SpanShape sh, LayerKv kv, RowMap rows, int t0, int tokens, int kr, int vr, __half* __restrict__ k16, __half* __restrict__ v16) {
+  pdl_enter();
+  const GroupKeys gk = group_keys(row_position(rows, t0), tokens, sh.window, sh.keep_first);
+  const int m = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, head = blockIdx.y, seq = row_sequence(rows, t0);
+  if (m >= gk.n) return;
+  auto put = [&](const float* src, int d, __half* dst, int w) {
+    for (int i = 4 * lane; i < w; i += 128) {
+      const float4 v = i < d ? *(const float4*)(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);  // d is a multiple of four
+      *(uint2*)(dst + i) = make_uint2(pack_h2(sat16(v.x), sat16(v.y)), pack_h2(sat16(v.z), sat16(v.w)));
+    }
+  };
+  const int j = gk.at(m);
+  put(kv.k + slot_of(kv, seq, j, kv.k_block, head, sh.dk), sh.dk, k16 + ((int64_t)head * gk.n + m) * kr, kr);
+  if (vr) put(kv.v + slot_of(kv, seq, j, kv.v_block, head, sh.dv), sh.dv, v16 + ((int64_t)head * gk.n + m) * vr, vr);
 }
 
 template <int ND, int NS>
 __global__ void __launch_bounds__(128 * NS)
-span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv kv, RowMap rows, int t0, int tokens, float* __restrict__ out,
-                __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate, int64_t gate_ld) {
+span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, const __half* __restrict__ k16, const __half* __restrict__ v16, bool shared_kv,
+                RowMap rows, int t0, int tokens, float* __restrict__ out, __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate,
+                int64_t gate_ld) {
   pdl_enter();
   constexpr int THR = 128 * NS, NT = CH / 8 / NS;  // score tiles of eight keys per warp
   static_assert(NT % 2 == 0, "keys are loaded sixteen at a time");
   extern __shared__ __align__(16) unsigned char raw[];
-  const MmaLayout L = mma_layout(sh.dk, sh.dv, ND, NS, kv.k == kv.v);
+  const MmaLayout L = mma_layout(sh.dk, sh.dv, ND, NS, shared_kv);
   __half* sq = (__half*)raw;
-  __half* sk = sq + 64 * L.qp;
-  __half* sv = L.shared ? sk : sk + CH * L.kp;
-  __half* sp = sk + CH * L.kp + (L.shared ? 0 : CH * L.vp);  // exponentials, NS > 1
+  __half* sk = sq + 64 * L.qp;                                         // keys (two buffers where they are the values)
+  __half* sv = sk + CH * L.kp;                                         // values, or the second buffer
+  __half* sp = sv + CH * L.vp;                                         // exponentials, NS > 1
   __shared__ float s_scale[64], s_red[NS][64];
-  __shared__ int64_t s_k[2][CH], s_v[2][CH];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
   const int rw = warp & 3, ns = warp >> 2;  // rows 16 rw .., key and value share ns
-  const int head = blockIdx.y, gq = sh.n_head / sh.n_kv, pairs = tokens * gq, pair0 = blockIdx.x * 64;
-  const int seq = row_sequence(rows, t0), p_first = row_position(rows, t0);
+  // the last rows first: in a window that is still filling they see the most keys
+  const int head = blockIdx.y, gq = sh.n_head / sh.n_kv, pairs = tokens * gq, pair0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 64;
+  const int p_first = row_position(rows, t0);
+  const GroupKeys gk = group_keys(p_first, tokens, sh.window, sh.keep_first);
   const int pa = p_first + pair0 / gq, pb = p_first + min(pairs - 1, pair0 + 63) / gq;  // positions of the tile's rows
   const int lo = sh.window > 0 ? max(0, pa - sh.window + 1) : 0, nk = min(sh.keep_first, lo), n_keys = nk + pb - lo + 1;
+  k16 += (int64_t)head * gk.n * L.kr;
+  v16 += (int64_t)head * gk.n * L.vr;
 
-  auto offsets = [&](int c, int buf) {  // where the keys of chunk c lie
-    if (tid < CH) {
-      const int m = c * CH + tid;
-      int64_t ko = -1, vo = -1;
-      if (m < n_keys) {
-        const int j = m < nk ? m : lo + m - nk;
-        ko = slot_of(kv, seq, j, kv.k_block, head, sh.dk);
-        vo = slot_of(kv, seq, j, kv.v_block, head, sh.dv);
-      }
-      s_k[buf][tid] = ko;
-      s_v[buf][tid] = vo;
+  // rows c * CH .. of the tile's own list; rows behind its end repeat the last one (their exponentials are zero)
+  auto stage = [&](__half* dst, const __half* src, int width, int pitch, int c) {
+    for (int p = tid >> 4; p < CH; p += THR / 16) {
+      const int m = min(c * CH + p, n_keys - 1);
+      const __half* row = src + (int64_t)gk.index(m < nk ? m : lo + m - nk) * width;
+      for (int d = 8 * (tid & 15); d < width; d += 128) copy16(dst + p * pitch + d, row + d);
     }
   };
+  stage(sk, k16, L.kr, L.kp, 0);
+  copy_commit();
   // queries: a warp per pair; the power of two that brings the largest magnitude into [2^9, 2^10)
   for (int r = warp; r < 64; r += 4 * NS) {
     const int p = pair0 + r;
@@ -390,18 +503,16 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
     for (int i = lane; i < L.kw; i += 32) sq[r * L.qp + i] = __float2half_rn(live && i < sh.dk ? sat16(src[i] * up) : 0.f);
     if (lane == 0) s_scale[r] = down * sh.scale;
   }
-  // padding columns of the key and value tiles are zero and stay so
-  for (int i = tid; i < CH * (L.kp - 8 - sh.dk); i += THR) sk[(i / (L.kp - 8 - sh.dk)) * L.kp + sh.dk + i % (L.kp - 8 - sh.dk)] = __float2half_rn(0.f);
-  if (!L.shared)
-    for (int i = tid; i < CH * (L.vw - sh.dv); i += THR) sv[(i / (L.vw - sh.dv)) * L.vp + sh.dv + i % (L.vw - sh.dv)] = __float2half_rn(0.f);
-  offsets(0, 0);
   __syncthreads();
 
+  constexpr float LOG2E = 1.4426950408889634f;  // scores are kept in units of ln 2: exp(x) = exp2(x log2 e)
   const int r0 = 16 * rw + g, r1 = r0 + 8;
   const int i0 = p_first + min(pair0 + r0, pairs - 1) / gq, i1 = p_first + min(pair0 + r1, pairs - 1) / gq;  // positions of this thread's rows
+  const int i_lo = p_first + min(pair0 + 16 * rw, pairs - 1) / gq, i_hi = p_first + min(pair0 + 16 * rw + 15, pairs - 1) / gq;  // of this warp's
   const float* b0 = sh.bias ? sh.bias + (int64_t)(head * gq + min(pair0 + r0, pairs - 1) % gq) * sh.bias_len : nullptr;
   const float* b1 = sh.bias ? sh.bias + (int64_t)(head * gq + min(pair0 + r1, pairs - 1) % gq) * sh.bias_len : nullptr;
-  const float f0 = s_scale[r0], f1 = s_scale[r1];
+  const float far0 = b0 ? b0[sh.bias_len - 1] * LOG2E : 0.f, far1 = b1 ? b1[sh.bias_len - 1] * LOG2E : 0.f;
+  const float f0 = s_scale[r0] * LOG2E, f1 = s_scale[r1] * LOG2E;
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
   float o[ND][4];
 #pragma unroll
@@ -415,29 +526,17 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
   };
   const int chunks = (n_keys + CH - 1) / CH;
   for (int c = 0; c < chunks; ++c) {
-    const int buf = c & 1;
-    {
-      const int kv4 = sh.dk / 4;
-      for (int i = tid; i < CH * kv4; i += THR) {
-        const int p = i / kv4, d = 4 * (i % kv4);
-        const int64_t off = s_k[buf][p];
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (off >= 0) v = *(const float4*)(kv.k + off + d);
-        *(uint2*)(sk + p * L.kp + d) = make_uint2(pack_h2(sat16(v.x), sat16(v.y)), pack_h2(sat16(v.z), sat16(v.w)));
-      }
-      if (!L.shared) {
-        const int vv4 = sh.dv / 4;
-        for (int i = tid; i < CH * vv4; i += THR) {
-          const int p = i / vv4, d = 4 * (i % vv4);
-          const int64_t off = s_v[buf][p];
-          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (off >= 0) v = *(const float4*)(kv.v + off + d);
-          *(uint2*)(sv + p * L.vp + d) = make_uint2(pack_h2(sat16(v.x), sat16(v.y)), pack_h2(sat16(v.z), sat16(v.w)));
-        }
-      }
+    __half* kt = L.shared && (c & 1) ? sv : sk;
+    __half* vt = L.shared ? kt : sv;
+    if (L.shared) {
+      if (c + 1 < chunks) { stage((c & 1) ? sk : sv, k16, L.kr, L.kp, c + 1); copy_commit(); copy_wait<1>(); }
+      else copy_wait<0>();
+    } else {
+      stage(sv, v16, L.vr, L.vp, c);
+      copy_commit();
+      copy_wait<1>();  // the keys
     }
     __syncthreads();
-    if (c + 1 < chunks) offsets(c + 1, buf ^ 1);
     // ---- scores of this warp's keys
     float s[NT][4];
 #pragma unroll
@@ -445,7 +544,7 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
 #pragma unroll
       for (int i = 0; i < 4; ++i) s[nt][i] = 0.f;
     const __half* qa = sq + (16 * rw + (lane & 15)) * L.qp + (lane >> 4) * 8;
-    const __half* kb = sk + (ns * 8 * NT + (lane & 7) + (lane >> 4) * 8) * L.kp + ((lane >> 3) & 1) * 8;
+    const __half* kb = kt + (ns * 8 * NT + (lane & 7) + (lane >> 4) * 8) * L.kp + ((lane >> 3) & 1) * 8;
 #pragma unroll 2
     for (int k0 = 0; k0 < L.kw; k0 += 16) {
       uint32_t a[4];
@@ -458,22 +557,32 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
         mma_f16(s[nt + 1], a, b[2], b[3]);
       }
     }
+    // this warp's keys of the chunk: positions between j_lo and j_hi (ascending list)
+    const int k_lo = c * CH + ns * 8 * NT, k_hi = k_lo + 8 * NT - 1;
+    const int j_lo = k_lo < nk ? k_lo : lo + k_lo - nk, j_hi = k_hi < nk ? k_hi : lo + k_hi - nk;
+    const bool all_seen = k_hi < n_keys && j_hi <= i_lo && (sh.window <= 0 || i_hi - j_lo < sh.window || j_hi < sh.keep_first);
+    const bool all_far = i_lo - j_hi >= sh.bias_len - 1;
     float x0 = -CUDART_INF_F, x1 = -CUDART_INF_F;
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
-        const int m = c * CH + ns * 8 * NT + 8 * nt + 2 * t4 + i, j = m < nk ? m : lo + m - nk;
-        const bool any = m < n_keys, kept = j < sh.keep_first || sh.window <= 0;
-        float u0 = s[nt][i] * f0, u1 = s[nt][2 + i] * f1;
-        const int d0 = i0 - j, d1 = i1 - j;
-        const bool v0 = any && d0 >= 0 && (kept || d0 < sh.window), v1 = any && d1 >= 0 && (kept || d1 < sh.window);
-        if (b0 && v0) u0 += __ldg(b0 + min(d0, sh.bias_len - 1));
-        if (b1 && v1) u1 += __ldg(b1 + min(d1, sh.bias_len - 1));
-        s[nt][i] = v0 ? u0 : -CUDART_INF_F;
-        s[nt][2 + i] = v1 ? u1 : -CUDART_INF_F;
-        x0 = fmaxf(x0, s[nt][i]);
-        x1 = fmaxf(x1, s[nt][2 + i]);
+        const int m = k_lo + 8 * nt + 2 * t4 + i, j = m < nk ? m : lo + m - nk;
+        float u0 = fmaf(s[nt][i], f0, far0), u1 = fmaf(s[nt][2 + i], f1, far1);
+        if (!all_far || !all_seen) {  // warp-uniform
+          const int d0 = i0 - j, d1 = i1 - j;
+          if (b0 && !all_far) {
+            u0 = fmaf(s[nt][i], f0, __ldg(b0 + min(max(d0, 0), sh.bias_len - 1)) * LOG2E);
+            u1 = fmaf(s[nt][2 + i], f1, __ldg(b1 + min(max(d1, 0), sh.bias_len - 1)) * LOG2E);
+          }
+          const bool any = m < n_keys, kept = j < sh.keep_first || sh.window <= 0;
+          if (!(any && d0 >= 0 && (kept || d0 < sh.window))) u0 = -CUDART_INF_F;
+          if (!(any && d1 >= 0 && (kept || d1 < sh.window))) u1 = -CUDART_INF_F;
+        }
+        s[nt][i] = u0;
+        s[nt][2 + i] = u1;
+        x0 = fmaxf(x0, u0);
+        x1 = fmaxf(x1, u1);
       }
     x0 = fmaxf(x0, __shfl_xor_sync(~0u, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(~0u, x0, 2));
     x1 = fmaxf(x1, __shfl_xor_sync(~0u, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(~0u, x1, 2));
@@ -485,9 +594,11 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
     }
     x0 = fmaxf(x0, m0);
     x1 = fmaxf(x1, m1);
-    const float w0 = m0 == -CUDART_INF_F ? 0.f : expf(m0 - x0), w1 = m1 == -CUDART_INF_F ? 0.f : expf(m1 - x1);
+    const float w0 = m0 == -CUDART_INF_F ? 0.f : exp2f(m0 - x0), w1 = m1 == -CUDART_INF_F ? 0.f : exp2f(m1 - x1);
     m0 = x0;
     m1 = x1;
+    // a row that has seen nothing yet: every score is -inf and so is the maximum; its exponentials are zero
+    const float c0 = m0 == -CUDART_INF_F ? 0.f : m0, c1 = m1 == -CUDART_INF_F ? 0.f : m1;
     l0 *= w0;
     l1 *= w1;
 #pragma unroll
@@ -495,14 +606,8 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
     uint32_t e0[NT], e1[NT];
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
-      float e[4];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        e[i] = s[nt][i] == -CUDART_INF_F ? 0.f : expf(s[nt][i] - m0);
-        e[2 + i] = s[nt][2 + i] == -CUDART_INF_F ? 0.f : expf(s[nt][2 + i] - m1);
-      }
-      e0[nt] = pack_h2(e[0], e[1]);
-      e1[nt] = pack_h2(e[2], e[3]);
+      e0[nt] = pack_h2(exp2f(s[nt][0] - c0), exp2f(s[nt][1] - c0));
+      e1[nt] = pack_h2(exp2f(s[nt][2] - c1), exp2f(s[nt][3] - c1));
       const __half2 h0 = *(const __half2*)&e0[nt], h1 = *(const __half2*)&e1[nt];
       l0 += __low2float(h0) + __high2float(h0);  // the sum of what the weighted sum below uses
       l1 += __low2float(h1) + __high2float(h1);
@@ -512,8 +617,13 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
       }
     }
     if constexpr (NS > 1) row_group();
+    if (!L.shared) {
+      copy_wait<0>();   // the values
+      __syncthreads();  // everyone's, and every warp is done with the keys
+      if (c + 1 < chunks) { stage(sk, k16, L.kr, L.kp, c + 1); copy_commit(); }
+    }
     // ---- weighted values: this warp's dimensions over all keys of the chunk
-    const __half* vb = sv + (lane & 15) * L.vp + ns * 8 * ND + (lane >> 4) * 8;
+    const __half* vb = vt + (lane & 15) * L.vp + ns * 8 * ND + (lane >> 4) * 8;
 #pragma unroll
     for (int k0 = 0; k0 < CH; k0 += 16) {
       uint32_t a[4];
@@ -530,7 +640,7 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, LayerKv
         mma_f16(o[nd + 1], a, b[2], b[3]);
       }
     }
-    __syncthreads();  // the next chunk overwrites the tiles
+    __syncthreads();  // the next copies overwrite the values
   }
   l0 += __shfl_xor_sync(~0u, l0, 1); l0 += __shfl_xor_sync(~0u, l0, 2);
   l1 += __shfl_xor_sync(~0u, l1, 1); l1 += __shfl_xor_sync(~0u, l1, 2);
@@ -670,7 +780,14 @@ size_t span_smem(const SpanShape& sh) {
 constexpr size_t SCRATCH_FLOATS = 16u << 20;
 int span_rows_per_pass(const SpanShape& sh) { return (int)std::min<size_t>(512, std::max<size_t>(1, SCRATCH_FLOATS / span_row_floats(sh))); }
 
-typedef void (*MmaKernel)(const float*, int64_t, SpanShape, LayerKv, RowMap, int, int, float*, __nv_bfloat16*, const float*, int64_t);
+// most keys a group of consecutive rows sees
+int span_group_keys(const SpanShape& sh, int rows) {
+  return sh.window > 0 ? (int)std::min<int64_t>(sh.n_ctx, (int64_t)sh.window + sh.keep_first + rows) : sh.n_ctx;
+}
+constexpr size_t MMA_SMEM_LIMIT = 222 * 1024;
+
+typedef void (*MmaKernel)(const float*, int64_t, SpanShape, const __half*, const __half*, bool, RowMap, int, int, float*, __nv_bfloat16*, const float*,
+                          int64_t);
 // the smallest instantiation that covers the value dimensions
 MmaKernel mma_kernel(int dv, int* nd, int* ns) {
 #define LLR_SPAN(N, S) if (dv <= 8 * N * S) { *nd = N; *ns = S; return span_mma_kernel<N, S>; }
@@ -693,14 +810,14 @@ cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float
                              const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
-  return launch_walk(qkv_store_kernel, dim3(tokens), dim3(512), 0, s, proj, ld, bias, q_norm, k_norm, sh, kv, rows);
+  return launch_walk(qkv_store_kernel, dim3(tokens), dim3(PROJ_THREADS), 0, s, proj, ld, bias, q_norm, k_norm, sh, kv, rows);
 }
 
 cudaError_t launch_latent_store(const float* proj, int ld, const float* w, int n, float eps, const LayerKv& kv, const RowMap& rows, int tokens,
                                 cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
-  return launch_walk(latent_store_kernel, dim3(tokens), dim3(256), 0, s, proj, ld, w, n, eps, kv, rows);
+  return launch_walk(latent_store_kernel, dim3(tokens), dim3(PROJ_THREADS), 0, s, proj, ld, w, n, eps, kv, rows);
 }
 
 cudaError_t launch_rows_bf16(const float* x, int64_t ld, int n, void* out16, int tokens, cudaStream_t s, uint64_t* launches) {
@@ -741,26 +858,41 @@ bool span_supported(const SpanShape& sh) {
   return sh.n_head > 0 && sh.n_kv > 0 && sh.n_head % sh.n_kv == 0 && sh.dk > 0 && sh.dv > 0 && sh.dv <= MAX_VALUE && sh.dk <= 1024 && sh.n_head <= 4096 &&
          span_smem(sh) <= 200 * 1024;
 }
-size_t span_scratch_floats(const SpanShape& sh) { return (size_t)span_rows_per_pass(sh) * span_row_floats(sh); }
+size_t span_scratch_floats(const SpanShape& sh, int max_rows) {
+  int nd = 0, ns = 0;
+  size_t gathered = 0;  // binary16 keys and values of one group
+  if (mma_kernel(sh.dv, &nd, &ns)) {
+    const MmaLayout L = mma_layout(sh.dk, sh.dv, nd, ns, false);  // not shared: the larger of the two
+    gathered = (size_t)sh.n_kv * span_group_keys(sh, max_rows) * (L.kr + L.vr) / 2 + 64;
+  }
+  return std::max((size_t)span_rows_per_pass(sh) * span_row_floats(sh), gathered);
+}
 
 cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape& sh, const LayerKv& kv, const RowMap& rows, int t0, int tokens,
                                   float* out, void* out16, const float* gate, int64_t gate_ld, float* scratch, bool tensor_cores, bool one_sequence,
-                                  cudaStream_t s, uint64_t* launches) {
+                                  const NewToken* nt, cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (!span_supported(sh)) return cudaErrorInvalidValue;
   const int gq = sh.n_head / sh.n_kv;
   if (tensor_cores && one_sequence && sh.dk % 8 == 0 && sh.dv % 8 == 0 && q_ld % 4 == 0 && gate_ld % 2 == 0 && ((uintptr_t)gate & 7) == 0) {
     int nd = 0, ns = 0;
     MmaKernel kern = mma_kernel(sh.dv, &nd, &ns);
-    const size_t smem = kern ? mma_smem(mma_layout(sh.dk, sh.dv, nd, ns, kv.k == kv.v), ns) : 0;
-    if (kern && smem <= 200 * 1024) {
+    const bool shared = kv.k == kv.v;
+    const MmaLayout L = mma_layout(sh.dk, sh.dv, nd, ns, shared);
+    const size_t smem = kern ? mma_smem(L, ns) : 0;
+    if (kern && smem <= MMA_SMEM_LIMIT) {
       if (smem > 40 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
       }
-      if (launches) ++*launches;
-      return launch_walk(kern, dim3((unsigned)(((int64_t)tokens * gq + 63) / 64), sh.n_kv), dim3(128 * ns), smem, s, q, q_ld, sh, kv, rows, t0, tokens, out,
-                         (__nv_bfloat16*)out16, gate, gate_ld);
+      if (launches) *launches += 2;
+      const int keys = span_group_keys(sh, tokens);
+      __half* k16 = (__half*)scratch;
+      __half* v16 = shared ? k16 : k16 + (size_t)sh.n_kv * keys * L.kr;
+      cudaError_t e = launch_walk(span_gather_kernel, dim3((keys + 7) / 8, sh.n_kv), dim3(256), 0, s, sh, kv, rows, t0, tokens, L.kr, L.vr, k16, v16);
+      if (e != cudaSuccess) return e;
+      return launch_walk(kern, dim3((unsigned)(((int64_t)tokens * gq + 63) / 64), sh.n_kv), dim3(128 * ns), smem, s, q, q_ld, sh, (const __half*)k16,
+                         (const __half*)v16, shared, rows, t0, tokens, out, (__nv_bfloat16*)out16, gate, gate_ld);
     }
   }
   const int groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA, chunk = span_chunk(sh), splits = span_splits(sh), per = span_rows_per_pass(sh);
@@ -773,9 +905,10 @@ cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape&
   for (int r = 0; r < tokens; r += per) {
     const int n = std::min(per, tokens - r);
     if (launches) *launches += 2;
-    cudaError_t e = launch_walk(kern, dim3(sh.n_kv * groups, splits, n), dim3(ATT_THREADS), smem, s, q, q_ld, sh, kv, rows, t0 + r, chunk, scratch);
+    cudaError_t e = launch_walk(kern, dim3(sh.n_kv * groups, splits, n), dim3(ATT_THREADS), smem, s, q, q_ld, sh, kv, rows, t0 + r, chunk, scratch,
+                                nt && tokens == 1 ? *nt : NewToken{});
     if (e != cudaSuccess) return e;
-    e = launch_walk(span_combine_kernel, dim3(sh.n_head, n), dim3(128), 0, s, (const float*)scratch, sh, rows, t0 + r, chunk, splits, out,
+    e = launch_walk(span_combine_kernel, dim3(sh.n_head, n, (sh.dv + 127) / 128), dim3(128), 0, s, (const float*)scratch, sh, rows, t0 + r, chunk, splits, out,
                     (__nv_bfloat16*)out16, gate, gate_ld);
     if (e != cudaSuccess) return e;
   }

@@ -148,6 +148,7 @@ struct llr_exec {
   bool limit_resolved = false;
   size_t limit = 0;
   std::unordered_set<llr_matrix*> live;
+  std::unordered_set<llr_session*> sessions;  // what they hold on the device goes with the executor
 };
 
 namespace {
@@ -466,6 +467,8 @@ cudaError_t launch_matmul(const MatView& m, const float* x, float* y, int64_t to
 
 }  // namespace llr
 
+namespace { void session_orphan(llr_session* s); }
+
 extern "C" {
 
 int llr_exec_create(int device, llr_exec** out) {
@@ -540,6 +543,7 @@ int llr_exec_destroy(llr_exec* e) {
   if (!e) return LLR_OK;
   DeviceGuard guard(e->device);
   cudaStreamSynchronize(e->stream);
+  for (llr_session* s : e->sessions) session_orphan(s);
   drop_all_cached(e);
   for (llr_matrix* m : e->live) {  // handles the caller still holds: free the device side
     cudaFree(m->dev);
@@ -1594,7 +1598,40 @@ int llr_program_free(llr_program* p) {
 }
 
 // ---------------------------------------------------------------- device-resident Llama walk
-namespace { struct LayeredDecoder; }
+namespace {
+// A decoder described layer by layer, as its session holds it (llr_layered.cuh has the functions).
+struct LayeredDecoder {
+  struct Layer {
+    llr_mixer mx{};
+    llr_mlp mlp{};
+    SpanShape span{};
+    int in_rows = 0, q_rows = 0, gate_col = 0;  // gate_col: where the gate rows start in a row of the stacked projection
+    int64_t k_off = 0, v_off = 0;               // floats into a pool block (a layer that reads another's latents: that layer's)
+    bool own_kv = true;
+    float *in_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *kv_norm = nullptr, *bias = nullptr, *mixer_norm = nullptr, *mlp_norm = nullptr;
+    void* up_k_t = nullptr;  // up_k with a head's rows and columns exchanged, for the tensor cores
+    // products whose operands the tensor cores take
+    bool tc_in = false, tc_out = false, tc_gu = false, tc_down = false, tc_up = false;
+  };
+  std::vector<Layer> layers;
+  float embd_scale = 1.f, eps = 0.f;
+  const llr_matrix *token_embd = nullptr, *pos_embd = nullptr;
+  size_t block_floats = 0, y_rows = 1;
+  float *proj = nullptr, *lat_q = nullptr, *lat_o = nullptr, *att = nullptr, *gu = nullptr, *act = nullptr, *y = nullptr, *scratch = nullptr;
+  void *x16 = nullptr, *a16 = nullptr, *b16 = nullptr;
+  ~LayeredDecoder() {
+    for (Layer& L : layers) {
+      float* p[] = {L.in_bias, L.q_norm, L.k_norm, L.kv_norm, L.bias, L.mixer_norm, L.mlp_norm};
+      for (float* q : p) if (q) cudaFree(q);
+      if (L.up_k_t) cudaFree(L.up_k_t);
+    }
+    float* p[] = {proj, lat_q, lat_o, att, gu, act, y, scratch};
+    for (float* q : p) if (q) cudaFree(q);
+    void* v[] = {x16, a16, b16};
+    for (void* q : v) if (q) cudaFree(q);
+  }
+};
+}  // namespace
 
 struct llr_session {
   llr_exec* owner = nullptr;
@@ -1667,7 +1704,13 @@ void session_release(llr_session* s) {
   for (llr::Program* p : s->gateup_prog) program_destroy(p);
   for (llr::Program* p : s->moe_gateup_prog) program_destroy(p);
   for (llr::Program* p : s->moe_down_prog) program_destroy(p);
+  s->dec.reset();
   cudaGetLastError();
+}
+// its executor goes: the handle stays the caller's, every later call on it fails
+void session_orphan(llr_session* s) {
+  session_release(s);
+  s->owner = nullptr;
 }
 
 cudaError_t session_matmul(llr_exec* e, const llr_matrix* m, size_t tokens, const float* x, float* y) {
@@ -2078,6 +2121,7 @@ int session_create(llr_exec* e, const llr_llama_model* m, size_t n_seq, size_t k
     delete s;
     return fail_cuda(e, ce, "session buffers");
   }
+  e->sessions.insert(s);
   *out = s;
   return LLR_OK;
 }
@@ -2101,6 +2145,7 @@ int llr_session_free(llr_session* s) {
   if (s->owner) {
     DeviceGuard guard(s->owner->device);
     cudaStreamSynchronize(s->owner->stream);
+    s->owner->sessions.erase(s);
     session_release(s);
   }
   delete s;

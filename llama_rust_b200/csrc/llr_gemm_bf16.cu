@@ -264,12 +264,13 @@ cudaError_t launch_tiles(const Bf16Product& p, const Args& a, cudaStream_t strea
 constexpr int SMS = 148;
 int tiles_of(int tokens, int rows, int batch, int bn) { return ((tokens + BM - 1) / BM) * ((rows + bn - 1) / bn) * batch; }
 // Width of a tile: with many tiles the one of 160 .. 256 (a multiple of `step`, so that both halves of a gated tile are
-// whole boxes of eight-row groups) whose waves over the SMs cost least; otherwise 128 or 64.
+// whole eight-row groups) for which operand traffic and waves over the SMs together cost least -- measured, a tile costs
+// about as much through the bytes it loads as through the wave it takes part in; otherwise 128 or 64.
 int tile_width(int tokens, int rows, int batch, int step = 16) {
   if (tiles_of(tokens, rows, batch, 256) < 132) return rows > 64 ? 128 : 64;
   int best = 256, cost = 1 << 30;
   for (int bn = 256; bn >= 160; bn -= step) {
-    const int c = ((tiles_of(tokens, rows, batch, bn) + SMS - 1) / SMS) * (bn + 24);  // 24: what a tile costs besides its columns
+    const int tiles = tiles_of(tokens, rows, batch, bn), c = tiles * (BM + bn) / SMS + (tiles + SMS - 1) / SMS * (BM + 256);
     if (c < cost) { cost = c; best = bn; }
   }
   return best;

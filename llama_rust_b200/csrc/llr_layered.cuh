@@ -2,38 +2,6 @@
 // description, device copies and buffers, and the forward pass over a batch's rows.  The session around it -- sequences,
 // paged pool, batches, logits, greedy decode and its graph -- is the one of the Llama walk.
 
-struct LayeredDecoder {
-  struct Layer {
-    llr_mixer mx{};
-    llr_mlp mlp{};
-    SpanShape span{};
-    int in_rows = 0, q_rows = 0, gate_col = 0;  // gate_col: where the gate rows start in a row of the stacked projection
-    int64_t k_off = 0, v_off = 0;               // floats into a pool block (a layer that reads another's latents: that layer's)
-    bool own_kv = true;
-    float *in_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *kv_norm = nullptr, *bias = nullptr, *mixer_norm = nullptr, *mlp_norm = nullptr;
-    void* up_k_t = nullptr;  // up_k with a head's rows and columns exchanged, for the tensor cores
-    // products whose operands the tensor cores take
-    bool tc_in = false, tc_out = false, tc_gu = false, tc_down = false, tc_up = false;
-  };
-  std::vector<Layer> layers;
-  float embd_scale = 1.f, eps = 0.f;
-  const llr_matrix *token_embd = nullptr, *pos_embd = nullptr;
-  size_t block_floats = 0, y_rows = 1;
-  float *proj = nullptr, *lat_q = nullptr, *lat_o = nullptr, *att = nullptr, *gu = nullptr, *act = nullptr, *y = nullptr, *scratch = nullptr;
-  void *x16 = nullptr, *a16 = nullptr, *b16 = nullptr;
-  ~LayeredDecoder() {
-    for (Layer& L : layers) {
-      float* p[] = {L.in_bias, L.q_norm, L.k_norm, L.kv_norm, L.bias, L.mixer_norm, L.mlp_norm};
-      for (float* q : p) if (q) cudaFree(q);
-      if (L.up_k_t) cudaFree(L.up_k_t);
-    }
-    float* p[] = {proj, lat_q, lat_o, att, gu, act, y, scratch};
-    for (float* q : p) if (q) cudaFree(q);
-    void* v[] = {x16, a16, b16};
-    for (void* q : v) if (q) cudaFree(q);
-  }
-};
-
 bool bf16_operand(const llr_matrix* m) { return m->dtype == LLR_DTYPE_BF16 && gemm_bf16_supported(m->dev, m->rows, m->cols); }
 
 // bucket(n) for n = 0 .. bias_max; from bias_max on every distance is in the last one.  A value within 1e-9 of a whole
@@ -361,6 +329,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
     delete s;
     return fail_cuda(e, ce, "session buffers");
   }
+  e->sessions.insert(s);
   *out = s;
   return LLR_OK;
 }

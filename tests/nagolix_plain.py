@@ -31,6 +31,15 @@ def read_model(folder):
     return cfg, w
 
 
+def bf16_round(a):
+    """Nearest bfloat16 values (what the serving path feeds its products with)."""
+    return bf16_to_f64(f32_to_bf16(a).tobytes()).reshape(np.shape(a))
+
+
+def exact(a):
+    return a
+
+
 def sigmoid(z):
     return 1.0 / (1.0 + np.exp(-np.asarray(z, np.float64)))
 
@@ -69,27 +78,30 @@ def clamped_glu(g, u, limit):
     return g * sigmoid(1.702 * g) * (u + 1.0)
 
 
-def dense_ff(x, w, p, limit):
-    return clamped_glu(x @ w[p + "gate"].T, x @ w[p + "up"].T, limit) @ w[p + "down"].T
+def dense_ff(x, w, p, limit, cast=exact):
+    x = cast(x)
+    return cast(clamped_glu(x @ w[p + "gate"].T, x @ w[p + "up"].T, limit)) @ w[p + "down"].T
 
 
-def latent_of(h, w, p, eps):
-    return rms(h @ w[p + "dkv"].T, eps) * w[p + "dkv.norm"]
+def latent_of(h, w, p, eps, cast=exact):
+    return rms(cast(h) @ w[p + "dkv"].T, eps) * w[p + "dkv.norm"]
 
 
-def latent_attention(h, c, w, p, m):
+def latent_attention(h, c, w, p, m, cast=exact):
     n, H, d, dv = len(h), m["heads"], m["dim"], m["vdim"]
+    h, c = cast(h), cast(c)
     q = (h @ w[p + "q"].T).reshape(n, H, d)
     k = (c @ w[p + "uk"].T).reshape(n, H, d)
     v = (c @ w[p + "uv"].T).reshape(n, H, dv)
     s = np.einsum("ihd,jhd->hij", q, k) * m["scale"]
     s = np.where(visible(n, m["mask"]["size"], 0)[None], s, -np.inf)
     o = np.einsum("hij,jhd->ihd", softmax(s), v) * sigmoid(h @ w[p + "g"].T)[:, :, None]
-    return o.reshape(n, H * dv) @ w[p + "o"].T
+    return cast(o.reshape(n, H * dv)) @ w[p + "o"].T
 
 
-def biased_attention(h, w, p, m, eps):
+def biased_attention(h, w, p, m, eps, cast=exact):
     n, H, G, d, dv = len(h), m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    h = cast(h)
     q = rms(h @ w[p + "q"].T + w[p + "q.b"], eps) * w[p + "q.norm"]
     k = rms(h @ w[p + "k"].T + w[p + "k.b"], eps) * w[p + "k.norm"]
     v = h @ w[p + "v"].T + w[p + "v.b"]
@@ -102,11 +114,12 @@ def biased_attention(h, w, p, m, eps):
     s = s + by_distance[dist].transpose(2, 0, 1)
     s = np.where(visible(n, m["mask"]["size"], m["mask"]["keep_first"])[None], s, -np.inf)
     o = np.einsum("hij,jhd->ihd", softmax(s), v).reshape(n, H * dv)
-    return (o * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+    return cast(o * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
 
 
-def forward(cfg, w, tokens, stream=None):
-    """Logits [n, vocab] of one sequence; `stream` (a list) receives the residual stream after every layer."""
+def forward(cfg, w, tokens, stream=None, cast=exact):
+    """Logits [n, vocab] of one sequence; `stream` (a list) receives the residual stream after every layer.  cast: applied
+    to what enters a product (bf16_round: how much that rounding alone changes)."""
     eps = cfg["norm"]["eps"]
     x = embed(np.asarray(tokens), w["embed"], w["pos"], cfg["embedding"]["scale"])
     latents = {}
@@ -115,13 +128,13 @@ def forward(cfg, w, tokens, stream=None):
         if L["type"] == "latent_attention":
             src = m.get("kv_from")
             if src is None:
-                latents[i] = latent_of(x, w, p, eps)
-            y = latent_attention(x, latents[i if src is None else src], w, p, m)
+                latents[i] = latent_of(x, w, p, eps, cast)
+            y = latent_attention(x, latents[i if src is None else src], w, p, m, cast)
         else:
-            y = biased_attention(x, w, p, m, eps)
+            y = biased_attention(x, w, p, m, eps, cast)
         x = x + rms(y, eps) * (1.0 + w[f"l{i}.norm1"])
         if L["mlp"] is not None:
-            x = x + rms(dense_ff(x, w, f"l{i}.mlp.", L["mlp"]["limit"]), eps) * (1.0 + w[f"l{i}.norm2"])
+            x = x + rms(dense_ff(x, w, f"l{i}.mlp.", L["mlp"]["limit"], cast), eps) * (1.0 + w[f"l{i}.norm2"])
         if stream is not None:
             stream.append(x.copy())
-    return (rms(x, eps) * (1.0 + w["final.norm"])) @ w["embed"].T
+    return cast(rms(x, eps) * (1.0 + w["final.norm"])) @ w["embed"].T

@@ -467,9 +467,9 @@ cudaError_t launch_matmul(const MatView& m, const float* x, float* y, int64_t to
 
 }  // namespace llr
 
-namespace { void session_orphan(llr_session* s); }
-
 extern "C" {
+
+namespace { void session_orphan(llr_session* s); }
 
 int llr_exec_create(int device, llr_exec** out) {
   if (!out) { g_create_error = "null output pointer"; return LLR_ERR_INVALID; }

@@ -135,24 +135,30 @@ __device__ __forceinline__ void attend_slice(const KV& src, const float* sq, flo
   for (int n = 0; n < ND; ++n)
 #pragma unroll
     for (int g = 0; g < ATT_MAX_GQA; ++g) acc[n][g] = 0.f;
+  if (grp < P) {
+    // runs of eight positions go to the groups in turn: the split does not depend on the KV block size.  The eight
+    // value rows of a run are fetched before the first is used; the sums are formed in ascending position order.
+    for (int sb = s0 + 8 * grp; sb < s1; sb += 8 * P) {
+      float vv[ND][8];
 #pragma unroll
-  for (int n = 0; n < ND; ++n)
-    if (grp < P && i + n * ATT_THREADS < dv) {
-      // runs of eight positions go to the groups in turn: the split does not depend on the KV block size.  The eight
-      // value rows of a run are fetched before the first is used; the sums are formed in ascending position order.
-      for (int sb = s0 + 8 * grp; sb < s1; sb += 8 * P) {
-        float vv[8];
+      for (int j = 0; j < 8; ++j) {
+        const float* vrow = sb + j < s1 ? src.v(sb + j) : nullptr;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) vv[j] = sb + j < s1 ? src.v(sb + j)[i + n * ATT_THREADS] : 0.f;
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
-          if (sb + j < s1) {
-#pragma unroll
-            for (int g = 0; g < ATT_MAX_GQA; ++g)
-              if (g < gqa) acc[n][g] = fmaf(sc[g * max_chunk + (sb + j - s0)], vv[j], acc[n][g]);
-          }
+        for (int n = 0; n < ND; ++n) vv[n][j] = vrow && i + n * ATT_THREADS < dv ? vrow[i + n * ATT_THREADS] : 0.f;
       }
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (sb + j < s1) {
+#pragma unroll
+          for (int g = 0; g < ATT_MAX_GQA; ++g)
+            if (g < gqa) {
+              const float e = sc[g * max_chunk + (sb + j - s0)];
+#pragma unroll
+              for (int n = 0; n < ND; ++n) acc[n][g] = fmaf(e, vv[n][j], acc[n][g]);
+            }
+        }
     }
+  }
   __syncthreads();  // the scores are no longer needed: their space takes the groups' partial sums
   float* vsum = sc;  // [P][gqa][dv]
 #pragma unroll

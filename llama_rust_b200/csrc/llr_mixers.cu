@@ -184,7 +184,7 @@ head_product_t_kernel(const uint16_t* __restrict__ w, int heads, int rows, int c
   if (one) {
     const uint16_t* wh = w + (int64_t)h * rows * cols + c;
     const float* xh = x + (int64_t)t0 * x_ld + (int64_t)h * rows;
-#pragma unroll 8
+#pragma unroll (TT == 1 ? 16 : 8)
     for (int r = grp; r < rows; r += 4) {
       float w0, w1;
       if (pair) {
@@ -278,17 +278,27 @@ __device__ __forceinline__ Span span_of(int pos, int window, int keep_first) {
 struct KvSpan {
   const LayerKv& kv;
   const SpanShape& sh;
+  const int2* where;  // page and place in it of the slice's keys, looked up once
   Span span;
-  int seq, head, pos, h0;  // kv head, the row's position, first query head
-  __device__ __forceinline__ const float* k(int m) const { return kv.k + slot_of(kv, seq, span.at(m), kv.k_block, head, sh.dk); }
-  __device__ __forceinline__ const float* v(int m) const { return kv.v + slot_of(kv, seq, span.at(m), kv.v_block, head, sh.dv); }
+  int s0, head, pos, h0;  // first key of the slice, kv head, the row's position, first query head
+  __device__ __forceinline__ const float* k(int m) const {
+    const int2 w = where[m - s0];
+    return kv.k + w.x * kv.k_block + (int64_t)(head * kv.block_tokens + w.y) * sh.dk;
+  }
+  __device__ __forceinline__ const float* v(int m) const {
+    const int2 w = where[m - s0];
+    return kv.v + w.x * kv.v_block + (int64_t)(head * kv.block_tokens + w.y) * sh.dv;
+  }
   __device__ __forceinline__ float score(int g, int m, float dot) const {
     const float s = __fmul_rn(dot, sh.scale);
     return sh.bias ? __fadd_rn(s, sh.bias[(int64_t)(h0 + g) * sh.bias_len + min(pos - span.at(m), sh.bias_len - 1)]) : s;
   }
 };
 
-// grid (kv head x group of at most ATT_MAX_GQA query heads, slice of the visible keys, row)
+// Query heads of a kv head that share a block: eight, four where a head's query and value rows are long.
+inline __host__ __device__ int span_heads(const SpanShape& sh) { return sh.dk + sh.dv > 512 ? ATT_MAX_GQA / 2 : ATT_MAX_GQA; }
+
+// grid (kv head x group of span_heads query heads, slice of the visible keys, row)
 // With nt (a single decode token) the kernel also does what the store kernels do for that token: the query is biased and
 // normed as it is loaded, and the blocks whose slice holds the token's own position write its key and value (or its
 // latent) into the cache and read them back like any other; blocks that share a kv head write the same values.
@@ -299,9 +309,10 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
                     NewToken nt) {
   pdl_enter();
   __shared__ float red[2][32];
-  extern __shared__ float sm[];  // q [heads][dk] | scores [heads][chunk] or sums [P][heads][dv]
-  const int gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
-  const int head = blockIdx.x / groups, g0 = (blockIdx.x % groups) * ATT_MAX_GQA, heads = min(ATT_MAX_GQA, gq - g0);
+  extern __shared__ int2 smw[];  // pages [chunk] | q [heads][dk] | scores [heads][chunk] or sums [P][heads][dv]
+  float* sm = (float*)(smw + chunk);
+  const int gq = sh.n_head / sh.n_kv, per = span_heads(sh), groups = (gq + per - 1) / per;
+  const int head = blockIdx.x / groups, g0 = (blockIdx.x % groups) * per, heads = min(per, gq - g0);
   const int t = t0 + blockIdx.z, split = blockIdx.y, n_split = (int)gridDim.y, h0 = head * gq + g0;
   const int pos = row_position(rows, t);
   const Span span = span_of(pos, sh.window, sh.keep_first);
@@ -309,6 +320,10 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
   if (s0 >= span.n) return;
   float* sq = sm;
   float* sc = sq + heads * sh.dk;
+  for (int m = s0 + threadIdx.x; m < s1; m += ATT_THREADS) {
+    const int j = span.at(m);
+    smw[m - s0] = make_int2(kv.table[(int64_t)row_sequence(rows, t) * kv.max_blocks + j / kv.block_tokens], j % kv.block_tokens);
+  }
   if (nt.proj && !nt.latent) {
     const QkvShape qs{sh.n_head, sh.n_kv, sh.dk, sh.dv, nt.eps};
     const QkvRow r = qkv_row(nt.proj, (int)q_ld, nt.bias, nt.q_norm, nt.k_norm, qs, red);
@@ -325,8 +340,8 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
   }
   __syncthreads();
   // records: [row of the pass][query head][slice][dv + 2]; a group's heads follow each other n_split records apart
-  float* rec = part + (((int64_t)blockIdx.z * sh.n_kv * groups + blockIdx.x) * n_split + split) * ATT_MAX_GQA * (sh.dv + 2);
-  attend_slice<MAX_VALUE>(KvSpan{kv, sh, span, row_sequence(rows, t), head, pos, h0}, sq, sc, rec, s0, s1, chunk, sh.dk, sh.dv, heads);
+  float* rec = part + (((int64_t)blockIdx.z * sh.n_kv * groups + blockIdx.x) * n_split + split) * per * (sh.dv + 2);
+  attend_slice<MAX_VALUE>(KvSpan{kv, sh, smw, span, s0, head, pos, h0}, sq, sc, rec, s0, s1, chunk, sh.dk, sh.dv, heads);
 }
 
 // grid (query head, row, 128 dimensions): merges a head's slices (at most 32) and applies the element gate
@@ -335,10 +350,10 @@ span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, i
                     __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate, int64_t gate_ld) {
   pdl_enter();
   const int lane = threadIdx.x & 31, h = blockIdx.x, t = t0 + blockIdx.y;
-  const int gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
-  const int bx = (h / gq) * groups + (h % gq) / ATT_MAX_GQA, g = (h % gq) % ATT_MAX_GQA;
+  const int gq = sh.n_head / sh.n_kv, per = span_heads(sh), groups = (gq + per - 1) / per;
+  const int bx = (h / gq) * groups + (h % gq) / per, g = (h % gq) % per;
   const int used = (span_of(row_position(rows, t), sh.window, sh.keep_first).n + chunk - 1) / chunk;
-  const int64_t stride = (int64_t)ATT_MAX_GQA * (sh.dv + 2);
+  const int64_t stride = (int64_t)per * (sh.dv + 2);
   const float* base = part + ((int64_t)blockIdx.y * sh.n_kv * groups + bx) * n_split * stride + g * (sh.dv + 2);
   const float ms = lane < used ? base[lane * stride + sh.dv] : -CUDART_INF_F;
   const float m = warp_max(ms);
@@ -763,19 +778,19 @@ clamped_glu_kernel(const float* __restrict__ gu, GluShape sh, float* __restrict_
 }
 
 // ---- launch shapes of the attention kernels ---------------------------------------------------------------------------
-constexpr int MAX_VALUE = 512;
+constexpr int MAX_VALUE = 4 * ATT_THREADS;
 int span_visible(const SpanShape& sh) {
   return sh.window > 0 ? (int)std::min<int64_t>(sh.n_ctx, (int64_t)sh.window + sh.keep_first) : sh.n_ctx;
 }
 int span_chunk(const SpanShape& sh) { return std::max(32, (span_visible(sh) + 31) / 32); }
 int span_splits(const SpanShape& sh) { return (span_visible(sh) + span_chunk(sh) - 1) / span_chunk(sh); }
 size_t span_row_floats(const SpanShape& sh) {
-  const size_t gq = sh.n_head / sh.n_kv, groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA;
-  return sh.n_kv * groups * span_splits(sh) * ATT_MAX_GQA * (size_t)(sh.dv + 2);
+  const size_t gq = sh.n_head / sh.n_kv, per = span_heads(sh), groups = (gq + per - 1) / per;
+  return sh.n_kv * groups * span_splits(sh) * per * (size_t)(sh.dv + 2);
 }
 size_t span_smem(const SpanShape& sh) {
-  const size_t heads = std::min(ATT_MAX_GQA, sh.n_head / sh.n_kv), P = std::max(1, ATT_THREADS / sh.dv);
-  return (heads * sh.dk + std::max(heads * span_chunk(sh), P * heads * sh.dv)) * sizeof(float);
+  const size_t heads = std::min(span_heads(sh), sh.n_head / sh.n_kv), P = std::max(1, ATT_THREADS / sh.dv);
+  return span_chunk(sh) * sizeof(int2) + (heads * sh.dk + std::max(heads * span_chunk(sh), P * heads * sh.dv)) * sizeof(float);
 }
 constexpr size_t SCRATCH_FLOATS = 16u << 20;
 int span_rows_per_pass(const SpanShape& sh) { return (int)std::min<size_t>(512, std::max<size_t>(1, SCRATCH_FLOATS / span_row_floats(sh))); }
@@ -895,9 +910,9 @@ cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape&
                          (const __half*)v16, shared, rows, t0, tokens, out, (__nv_bfloat16*)out16, gate, gate_ld);
     }
   }
-  const int groups = (gq + ATT_MAX_GQA - 1) / ATT_MAX_GQA, chunk = span_chunk(sh), splits = span_splits(sh), per = span_rows_per_pass(sh);
+  const int groups = (gq + span_heads(sh) - 1) / span_heads(sh), chunk = span_chunk(sh), splits = span_splits(sh), per = span_rows_per_pass(sh);
   const size_t smem = span_smem(sh);
-  auto kern = sh.dv <= ATT_THREADS ? span_partial_kernel<ATT_THREADS> : span_partial_kernel<MAX_VALUE>;
+  auto kern = sh.dv <= ATT_THREADS ? span_partial_kernel<ATT_THREADS> : sh.dv <= 2 * ATT_THREADS ? span_partial_kernel<2 * ATT_THREADS> : span_partial_kernel<MAX_VALUE>;
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute((const void*)kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;

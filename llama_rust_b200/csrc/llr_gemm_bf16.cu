@@ -114,7 +114,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
   uint32_t* tmem_slot = (uint32_t*)(done + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int bn = a.bn, width = GLU ? bn / 2 : bn;  // results per activation row of the tile
-  const int row0 = blockIdx.x * width, tok0 = blockIdx.y * BM;
+  // token tiles run fastest: the CTAs that share weight rows run at the same time, and the weights are read from HBM once
+  const int row0 = blockIdx.y * width, tok0 = blockIdx.x * BM;
   const int z = (int)blockIdx.z / a.slices, slice = (int)blockIdx.z % a.slices;
   const int per = (a.nk + a.slices - 1) / a.slices, k0 = slice * per, k1 = min(a.nk, k0 + per);  // never empty: the launcher sees to it
 
@@ -256,7 +257,8 @@ cudaError_t launch_tiles(const Bf16Product& p, const Args& a, cudaStream_t strea
     if (e != cudaSuccess) return e;
     slot.store(1, std::memory_order_relaxed);
   }
-  const dim3 grid((unsigned)((p.rows + width - 1) / width), (unsigned)((p.tokens + BM - 1) / BM), (unsigned)(p.batch * a.slices));
+  const dim3 grid((unsigned)((p.tokens + BM - 1) / BM), (unsigned)((p.rows + width - 1) / width), (unsigned)(p.batch * a.slices));
+  if (grid.y > 65535 || grid.z > 65535) return cudaErrorInvalidValue;
   gemm_bf16_kernel<BN, GLU><<<grid, THREADS, smem, stream>>>(xmap, wmap, a, err);
   return cudaGetLastError();
 }
@@ -264,13 +266,14 @@ cudaError_t launch_tiles(const Bf16Product& p, const Args& a, cudaStream_t strea
 constexpr int SMS = 148;
 int tiles_of(int tokens, int rows, int batch, int bn) { return ((tokens + BM - 1) / BM) * ((rows + bn - 1) / bn) * batch; }
 // Width of a tile: with many tiles the one of 160 .. 256 (a multiple of `step`, so that both halves of a gated tile are
-// whole eight-row groups) for which operand traffic and waves over the SMs together cost least -- measured, a tile costs
-// about as much through the bytes it loads as through the wave it takes part in; otherwise 128 or 64.
+// whole eight-row groups) whose waves over the SMs cost least, where a wave costs as much as its columns and WAVE_COST
+// more (measured: it hardly depends on the width); otherwise 128 or 64.
+constexpr int WAVE_COST = 450;
 int tile_width(int tokens, int rows, int batch, int step = 16) {
   if (tiles_of(tokens, rows, batch, 256) < 132) return rows > 64 ? 128 : 64;
   int best = 256, cost = 1 << 30;
   for (int bn = 256; bn >= 160; bn -= step) {
-    const int tiles = tiles_of(tokens, rows, batch, bn), c = tiles * (BM + bn) / SMS + (tiles + SMS - 1) / SMS * (BM + 256);
+    const int c = (tiles_of(tokens, rows, batch, bn) + SMS - 1) / SMS * (bn + WAVE_COST);
     if (c < cost) { cost = c; best = bn; }
   }
   return best;

@@ -567,17 +567,17 @@ int llr_session_max_batch(const llr_session* session, size_t* rows);
  * the layer has an mlp: the sublayers read x itself.  norm(y) = y / sqrt(mean(y^2) + norm_eps) * w, w as given here.
  * logits = output (norm(x)).
  *
- * LLR_MIXER_ATTENTION: `in` stacks the rows q (n_head * dim) | k (n_head_kv * dim) | v (n_head_kv * vdim) | gate;
+ * LLR_MIXER_ATTENTION: in_proj stacks the rows q (n_head * dim) | k (n_head_kv * dim) | v (n_head_kv * vdim) | gate;
  *   in_bias (NULL: none) holds the q | k | v rows' biases; q_norm / k_norm (NULL: none) weigh an RMS norm over ALL rows
  *   of q / of k before they are split into heads.  score = (q . k) * scale + rel[bucket(distance)][head] when n_bucket > 0:
  *   with h = n_bucket / 2, bucket(n) = n for n < h, else min(n_bucket - 1, h + floor(ln(n / h) / ln(bias_max / h) *
  *   (n_bucket - h))).
- * LLR_MIXER_LATENT: `in` stacks q (n_head * dim) | latent (kv_rank) | gate; the latent, RMS-normed with kv_norm, is what
+ * LLR_MIXER_LATENT: in_proj stacks q (n_head * dim) | latent (kv_rank) | gate; the latent, RMS-normed with kv_norm, is what
  *   the cache holds; keys are up_k latent, values up_v latent (BF16 matrices n_head * dim / n_head * vdim x kv_rank, head by head).
- *   kv_from >= 0: no latent rows in `in`; the cached latents of that earlier latent layer are read instead.
+ *   kv_from >= 0: no latent rows in in_proj; the cached latents of that earlier latent layer are read instead.
  * Both: window > 0: position i sees j with i - j < window, or j < keep_first; window 0: every earlier position.
  *   LLR_GATE_ELEMENT (attention): the concatenated heads times sigmoid of n_head * vdim gate rows; LLR_GATE_HEAD (latent):
- *   each head times sigmoid of its gate row.  `out`: n_embd x n_head * vdim.
+ *   each head times sigmoid of its gate row.  out_proj: n_embd x n_head * vdim.
  * mlp: n_ff 0: none.  gate_up stacks gate | up (2 n_ff x n_embd); a = min(gate, limit), b = clamp(up, -limit, limit);
  *   y = down (a * sigmoid(alpha * a) * (b + shift)). */
 #define LLR_MIXER_ATTENTION 0
@@ -592,7 +592,7 @@ typedef struct llr_mixer {
   uint32_t gate;
   float scale;
   uint32_t n_bucket, bias_max;
-  const llr_matrix *in, *up_k, *up_v, *out;
+  const llr_matrix *in_proj, *up_k, *up_v, *out_proj;
   const float *in_bias, *q_norm, *k_norm, *kv_norm; /* host, copied */
   const float* rel;                                 /* host, n_bucket x n_head, copied */
 } llr_mixer;

@@ -82,7 +82,7 @@ class LlamaModel(C.Structure):
 class Mixer(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("kind", "n_head", "n_head_kv", "dim", "vdim", "kv_rank", "window", "keep_first")] + \
                [("kv_from", C.c_int32), ("gate", C.c_uint32), ("scale", C.c_float), ("n_bucket", C.c_uint32), ("bias_max", C.c_uint32)] + \
-               [(n, C.c_void_p) for n in ("in_", "up_k", "up_v", "out", "in_bias", "q_norm", "k_norm", "kv_norm", "rel")]
+               [(n, C.c_void_p) for n in ("in_proj", "up_k", "up_v", "out_proj", "in_bias", "q_norm", "k_norm", "kv_norm", "rel")]
 
 
 class Mlp(C.Structure):

@@ -55,7 +55,7 @@ std::string layered_check(llr_exec* e, const llr_decoder_model* m, size_t li, co
     return "unknown mixer";
   }
   if (!span_supported(L.span)) return "head sizes, latent size or context length outside the attention kernels";
-  if (!shape(x.in, (size_t)L.in_rows, E) || !shape(x.out, E, H * x.vdim)) return "in / out do not match the mixer's sizes";
+  if (!shape(x.in_proj, (size_t)L.in_rows, E) || !shape(x.out_proj, E, H * x.vdim)) return "in_proj / out_proj do not match the mixer's sizes";
   if (!D.mixer_norm || (D.mlp.n_ff > 0 && !D.mlp_norm)) return "a norm is missing";
   if (D.mlp.n_ff > 0 && (!shape(D.mlp.gate_up, 2 * (size_t)D.mlp.n_ff, E) || !shape(D.mlp.down, E, D.mlp.n_ff) || !(D.mlp.limit >= 0.f)))
     return "gate_up / down do not match n_ff, or the limit is negative";
@@ -95,7 +95,7 @@ cudaError_t layered_layers(llr_session* s, const int* ids_dev, size_t n, const R
     const bool latent = mx.kind == LLR_MIXER_LATENT, up_tc = tc && L.tc_up, out_tc = tc && L.tc_out;
     const LayerKv kv{s->cache_k + L.k_off, s->cache_k + L.v_off, s->table_dev, (int)s->block_tokens, (int)s->max_blocks, (int64_t)D.block_floats,
                      (int64_t)D.block_floats};
-    if ((ce = product(mx.in, tc && L.tc_in, s->x, D.x16, D.proj, nullptr)) != cudaSuccess) return ce;
+    if ((ce = product(mx.in_proj, tc && L.tc_in, s->x, D.x16, D.proj, nullptr)) != cudaSuccess) return ce;
     const float* gate = mx.gate != LLR_GATE_NONE ? D.proj + L.gate_col : nullptr;
     const float* q = D.proj;
     int64_t q_ld = L.in_rows;
@@ -167,7 +167,7 @@ cudaError_t layered_layers(llr_session* s, const int* ids_dev, size_t n, const R
       if (ce != cudaSuccess) return ce;
     }
     int slices = 1;
-    if ((ce = product(mx.out, out_tc, D.att, h16, D.y, &slices)) != cudaSuccess ||
+    if ((ce = product(mx.out_proj, out_tc, D.att, h16, D.y, &slices)) != cudaSuccess ||
         (ce = launch_norm_add(s->x, D.y, slices, (int64_t)n * E, L.mixer_norm, D.eps, tc ? D.x16 : nullptr, N, E, st, lc)) != cudaSuccess)
       return ce;
     if (L.mlp.n_ff == 0) continue;
@@ -236,8 +236,8 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
         D->block_floats += up4((size_t)L.span.n_kv * block_tokens * L.span.dv);
       }
     }
-    L.tc_in = bf16_operand(x.in);
-    L.tc_out = bf16_operand(x.out);
+    L.tc_in = bf16_operand(x.in_proj);
+    L.tc_out = bf16_operand(x.out_proj);
     L.tc_gu = L.mlp.n_ff > 0 && bf16_operand(L.mlp.gate_up);
     L.tc_down = L.mlp.n_ff > 0 && bf16_operand(L.mlp.down);
     const size_t H = x.n_head, R = x.kv_rank;
@@ -314,7 +314,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
   if (lat) { alloc(&D->lat_q, B * lat); alloc(&D->lat_o, B * lat); }
   if (ff) { alloc(&D->gu, B * 2 * ff); alloc(&D->act, B * ff); }
   for (const auto& L : D->layers)
-    for (const llr_matrix* w : {L.mx.out, L.mlp.n_ff > 0 ? L.mlp.down : L.mx.out})
+    for (const llr_matrix* w : {L.mx.out_proj, L.mlp.n_ff > 0 ? L.mlp.down : L.mx.out_proj})
       for (size_t n = 1; n <= B; ++n) D->y_rows = std::max(D->y_rows, n * (size_t)gemm_bf16_slices((int)n, (int)w->rows, (int)w->cols));
   alloc(&D->y, D->y_rows * E);
   alloc16(&D->x16, B * E); alloc16(&D->a16, B * a16); alloc16(&D->b16, B * b16);

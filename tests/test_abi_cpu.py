@@ -149,7 +149,8 @@ def test_ctypes_structures_have_the_layout_of_the_header(tmp_path):
         pytest.skip("no C compiler")
     pairs = {"llr_counters": _lib.Counters, "llr_gguf_tensor": _lib.GgufTensor, "llr_program_entry": _lib.ProgramEntry,
              "llr_program_op": _lib.ProgramOp, "llr_program_shard": _lib.ProgramShard, "llr_llama_config": _lib.LlamaConfig,
-             "llr_llama_layer": _lib.LlamaLayer, "llr_llama_model": _lib.LlamaModel, "llr_moe_layer": _lib.MoeLayer}
+             "llr_llama_layer": _lib.LlamaLayer, "llr_llama_model": _lib.LlamaModel, "llr_moe_layer": _lib.MoeLayer,
+             "llr_mixer": _lib.Mixer, "llr_mlp": _lib.Mlp, "llr_decoder_layer": _lib.DecoderLayer, "llr_decoder_model": _lib.DecoderModel}
     header = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "include", "llama_rust_b200.h")
     lines = ['#include <stdio.h>', '#include <stddef.h>', f'#include "{header}"', 'int main(void) {']
     for cname, st in pairs.items():

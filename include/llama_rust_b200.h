@@ -563,9 +563,9 @@ int llr_session_max_batch(const llr_session* session, size_t* rows);
  * on the tensor cores with bfloat16 activations, and prompt chunks of 16 rows and more run their attention with binary16
  * operands; norms, scores, softmax, gates and the residual stream are f32 either way.
  *
- * x = token_embd[token] * embd_scale (+ pos_embd[position]); per layer x += norm(mixer(x)), then x += norm(mlp(x)) when
- * the layer has an mlp: the sublayers read x itself.  norm(y) = y / sqrt(mean(y^2) + norm_eps) * w, w as given here.
- * logits = output (norm(x)).
+ * x = token_embd[token] * embd_scale (+ pos_embd[position]).  LLR_NORM_OUTPUT: per layer x += norm(mixer(x)), then x +=
+ * norm(mlp(x)) when the layer has an mlp.  LLR_NORM_INPUT: x += mixer(norm(x)), then x += mlp(norm(x)).
+ * norm(y) = y / sqrt(mean(y^2) + norm_eps) * w, w as given here.  logits = output (norm(x)).
  *
  * LLR_MIXER_ATTENTION: in_proj stacks the rows q (n_head * dim) | k (n_head_kv * dim) | v (n_head_kv * vdim) | gate;
  *   in_bias (NULL: none) holds the q | k | v rows' biases; q_norm / k_norm (NULL: none) weigh an RMS norm over ALL rows
@@ -576,12 +576,40 @@ int llr_session_max_batch(const llr_session* session, size_t* rows);
  *   the cache holds; keys are up_k latent, values up_v latent (BF16 matrices n_head * dim / n_head * vdim x kv_rank, head by head).
  *   kv_from >= 0: no latent rows in in_proj; the cached latents of that earlier latent layer are read instead.
  * Both: window > 0: position i sees j with i - j < window, or j < keep_first; window 0: every earlier position.
- *   LLR_GATE_ELEMENT (attention): the concatenated heads times sigmoid of n_head * vdim gate rows; LLR_GATE_HEAD (latent):
+ *   LLR_GATE_ELEMENT (attention): the concatenated heads times sigmoid of n_head * vdim gate rows; LLR_GATE_HEAD:
  *   each head times sigmoid of its gate row.  out_proj: n_embd x n_head * vdim.
- * mlp: n_ff 0: none.  gate_up stacks gate | up (2 n_ff x n_embd); a = min(gate, limit), b = clamp(up, -limit, limit);
- *   y = down (a * sigmoid(alpha * a) * (b + shift)). */
+ *   Attention: rot_dims > 0 rotates the first rot_dims values of each query and key head by its position (behind the norms):
+ *   pair (i, i + rot_dims / 2) by the angle position * rot_freq[i].  sink (NULL: none): exp(sink[h]) stands in the softmax's
+ *   denominator beside the keys.
+ * Recurrent mixers keep a state per sequence in f32 instead of cached positions:
+ * LLR_MIXER_RETENTION: in_proj stacks q (n_head * dim) | k (n_head * dim) | v (n_head * vdim) | gate (n_head * vdim); q and k
+ *   rotated as above; per head S = decay[h] S + (scale k) v^T, o = S^T q; o / rms(o) times silu(gate) enters out_proj.
+ * LLR_MIXER_DELTA: in_proj stacks q (n_head_kv * dim) | k (n_head_kv * dim) | v (n_head * vdim) | decay (decay_rank) | gate
+ *   (gate_rank) | beta (n_head).  q | k | v pass a causal convolution over `taps` rows per channel (conv: channels x taps, the
+ *   last tap weighs the row itself) and silu; q and k become unit vectors x / sqrt(sum x^2 + unit_eps), q times scale.
+ *   g = exp(-exp(decay[h]) softplus(decay_up (decay rows) + step_bias)), n_head x dim; beta = sigmoid.  Per head S = diag(g) S,
+ *   u = beta (v - S^T k), S += k u^T, o = S^T q; o / rms(o) * head_norm times sigmoid(gate_up (gate rows)) enters out_proj.
+ *   decay_up: BF16, n_head * dim x decay_rank; gate_up: BF16, n_head * vdim x gate_rank.
+ * LLR_MIXER_GATED_LINEAR: in_proj stacks y (width) | x (width), in_bias (NULL: none) their biases; u = convolution of x (conv, plus
+ *   conv_bias); per block of width / blocks channels r | i = sigmoid(gates u + gate_bias), gates a BF16 matrix that stacks
+ *   the blocks' r rows | i rows (2 width x width / blocks); log a = -scale r softplus(decay[c]); S = a S + sqrt(1 - a^2) i u;
+ *   S gelu(y) enters out_proj (n_embd x width).
+ * A layer may have a second mixer beside the first that reads the same input: `beside`, whose in_proj and out_proj are NULL.
+ *   The first one's in_proj then goes on with the second's rows from a multiple of eight rows on, its out_proj with the
+ *   second's columns; their results are multiplied by mixer_scale and beside_scale (which nothing reads otherwise).
+ *   in_proj may have more rows than its mixers need.
+ * A recurrent state cannot be rewound: such sessions take llr_session_seq_truncate to 0 or to the position itself only.
+ * mlp: n_ff 0: none.  gate_up stacks gate | up (2 n_ff x n_embd).  LLR_UNIT_CLAMPED: a = min(gate, limit), b = clamp(up, -limit,
+ *   limit), y = down (a * sigmoid(alpha * a) * (b + shift)); LLR_UNIT_GELU: y = down (gelu(gate) * up), gelu in its tanh form. */
 #define LLR_MIXER_ATTENTION 0
 #define LLR_MIXER_LATENT 1
+#define LLR_MIXER_RETENTION 2
+#define LLR_MIXER_DELTA 3
+#define LLR_MIXER_GATED_LINEAR 4
+#define LLR_NORM_OUTPUT 0
+#define LLR_NORM_INPUT 1
+#define LLR_UNIT_CLAMPED 0
+#define LLR_UNIT_GELU 1
 #define LLR_GATE_NONE 0
 #define LLR_GATE_ELEMENT 1
 #define LLR_GATE_HEAD 2
@@ -595,9 +623,16 @@ typedef struct llr_mixer {
   const llr_matrix *in_proj, *up_k, *up_v, *out_proj;
   const float *in_bias, *q_norm, *k_norm, *kv_norm; /* host, copied */
   const float* rel;                                 /* host, n_bucket x n_head, copied */
+  uint32_t rot_dims;
+  const double* rot_freq; /* host, rot_dims / 2, copied */
+  const float* sink;      /* host, n_head, copied */
+  uint32_t width, blocks, taps, decay_rank, gate_rank;
+  float unit_eps;
+  const llr_matrix *gates, *decay_up, *gate_up;
+  const float *conv, *conv_bias, *gate_bias, *decay, *step_bias, *head_norm; /* host, copied */
 } llr_mixer;
 typedef struct llr_mlp {
-  uint32_t n_ff;
+  uint32_t n_ff, unit;
   float limit, alpha, shift;
   const llr_matrix *gate_up, *down;
 } llr_mlp;
@@ -605,9 +640,11 @@ typedef struct llr_decoder_layer {
   llr_mixer mixer;
   llr_mlp mlp;
   const float *mixer_norm, *mlp_norm; /* host, n_embd floats, copied */
+  const llr_mixer* beside;            /* NULL: none */
+  float mixer_scale, beside_scale;
 } llr_decoder_layer;
 typedef struct llr_decoder_model {
-  uint32_t n_layer, n_embd, n_vocab, n_ctx;
+  uint32_t n_layer, n_embd, n_vocab, n_ctx, norm_place;
   float norm_eps, embd_scale;
   const llr_matrix* token_embd; /* BF16 */
   const llr_matrix* pos_embd;   /* BF16, at least n_ctx rows, or NULL */

@@ -82,20 +82,24 @@ class LlamaModel(C.Structure):
 class Mixer(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("kind", "n_head", "n_head_kv", "dim", "vdim", "kv_rank", "window", "keep_first")] + \
                [("kv_from", C.c_int32), ("gate", C.c_uint32), ("scale", C.c_float), ("n_bucket", C.c_uint32), ("bias_max", C.c_uint32)] + \
-               [(n, C.c_void_p) for n in ("in_proj", "up_k", "up_v", "out_proj", "in_bias", "q_norm", "k_norm", "kv_norm", "rel")]
+               [(n, C.c_void_p) for n in ("in_proj", "up_k", "up_v", "out_proj", "in_bias", "q_norm", "k_norm", "kv_norm", "rel")] + \
+               [("rot_dims", C.c_uint32), ("rot_freq", C.c_void_p), ("sink", C.c_void_p)] + \
+               [(n, C.c_uint32) for n in ("width", "blocks", "taps", "decay_rank", "gate_rank")] + [("unit_eps", C.c_float)] + \
+               [(n, C.c_void_p) for n in ("gates", "decay_up", "gate_up", "conv", "conv_bias", "gate_bias", "decay", "step_bias", "head_norm")]
 
 
 class Mlp(C.Structure):
-    _fields_ = [("n_ff", C.c_uint32), ("limit", C.c_float), ("alpha", C.c_float), ("shift", C.c_float),
+    _fields_ = [("n_ff", C.c_uint32), ("unit", C.c_uint32), ("limit", C.c_float), ("alpha", C.c_float), ("shift", C.c_float),
                 ("gate_up", C.c_void_p), ("down", C.c_void_p)]
 
 
 class DecoderLayer(C.Structure):
-    _fields_ = [("mixer", Mixer), ("mlp", Mlp), ("mixer_norm", C.c_void_p), ("mlp_norm", C.c_void_p)]
+    _fields_ = [("mixer", Mixer), ("mlp", Mlp), ("mixer_norm", C.c_void_p), ("mlp_norm", C.c_void_p), ("beside", C.POINTER(Mixer)),
+                ("mixer_scale", C.c_float), ("beside_scale", C.c_float)]
 
 
 class DecoderModel(C.Structure):
-    _fields_ = [(n, C.c_uint32) for n in ("n_layer", "n_embd", "n_vocab", "n_ctx")] + \
+    _fields_ = [(n, C.c_uint32) for n in ("n_layer", "n_embd", "n_vocab", "n_ctx", "norm_place")] + \
                [("norm_eps", C.c_float), ("embd_scale", C.c_float)] + \
                [(n, C.c_void_p) for n in ("token_embd", "pos_embd", "output", "output_norm")] + \
                [("layers", C.POINTER(DecoderLayer))]

@@ -1601,33 +1601,57 @@ int llr_program_free(llr_program* p) {
 namespace {
 // A decoder described layer by layer, as its session holds it (llr_layered.cuh has the functions).
 struct LayeredDecoder {
-  struct Layer {
+  struct Mixer {
     llr_mixer mx{};
-    llr_mlp mlp{};
     SpanShape span{};
-    int in_rows = 0, q_rows = 0, gate_col = 0;  // gate_col: where the gate rows start in a row of the stacked projection
-    int64_t k_off = 0, v_off = 0;               // floats into a pool block (a layer that reads another's latents: that layer's)
-    bool own_kv = true;
-    float *in_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *kv_norm = nullptr, *bias = nullptr, *mixer_norm = nullptr, *mlp_norm = nullptr;
-    void* up_k_t = nullptr;  // up_k with a head's rows and columns exchanged, for the tensor cores
+    int in_col = 0, in_rows = 0, q_rows = 0, gate_col = 0;  // where its rows and its gate rows start in a row of the stacked projection
+    int out_col = 0, out_cols = 0;                          // its columns of out_proj
+    float scale = 1.f;                                      // of its result
+    int64_t k_off = 0, v_off = 0;  // floats into a pool block (a layer that reads another's latents: that layer's)
+    bool own_kv = true, recurrent = false;
+    int64_t state_off = 0, tail_off = 0;  // floats into a sequence's state: the recurrence's, the convolution's last inputs
+    int rot_off = 0;                      // of its rotation in a row's angles
+    int channels = 0;                     // of the convolution
+    float *in_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr, *kv_norm = nullptr, *bias = nullptr, *sink = nullptr, *conv = nullptr,
+          *conv_bias = nullptr, *gate_bias = nullptr, *decay = nullptr, *step_bias = nullptr, *head_norm = nullptr;
+    void* up_k_t = nullptr;   // up_k with a head's rows and columns exchanged, for the tensor cores
+    void* gates3 = nullptr;   // gates with every block's columns three times, for the tensor cores
+    bool tc_up = false;       // the mixer's own products (latent space, gates, low-rank) as tensor-core products
+  };
+  struct Layer {
+    std::vector<Mixer> mixers;  // one, or two beside each other
+    llr_mlp mlp{};
+    const llr_matrix *in_proj = nullptr, *out_proj = nullptr;
+    float *mixer_norm = nullptr, *mlp_norm = nullptr;
     // products whose operands the tensor cores take
-    bool tc_in = false, tc_out = false, tc_gu = false, tc_down = false, tc_up = false;
+    bool tc_in = false, tc_out = false, tc_gu = false, tc_down = false;
   };
   std::vector<Layer> layers;
   float embd_scale = 1.f, eps = 0.f;
+  bool norm_input = false;
   const llr_matrix *token_embd = nullptr, *pos_embd = nullptr;
-  size_t block_floats = 0, y_rows = 1;
-  float *proj = nullptr, *lat_q = nullptr, *lat_o = nullptr, *att = nullptr, *gu = nullptr, *act = nullptr, *y = nullptr, *scratch = nullptr;
+  size_t block_floats = 0, y_rows = 1, state_floats = 0;
+  std::vector<double> freq;  // every distinct rotation, end to end
+  float *proj = nullptr, *lat_q = nullptr, *lat_o = nullptr, *att = nullptr, *gu = nullptr, *act = nullptr, *y = nullptr, *scratch = nullptr, *state = nullptr,
+        *prep = nullptr, *low = nullptr;  // low: what the mixers' own products leave
   void *x16 = nullptr, *a16 = nullptr, *b16 = nullptr;
+  double* freq_dev = nullptr;
+  float2* angles = nullptr;
+  int* group_first = nullptr;  // first row of each group of the batch in flight, and their end
   ~LayeredDecoder() {
     for (Layer& L : layers) {
-      float* p[] = {L.in_bias, L.q_norm, L.k_norm, L.kv_norm, L.bias, L.mixer_norm, L.mlp_norm};
-      for (float* q : p) if (q) cudaFree(q);
-      if (L.up_k_t) cudaFree(L.up_k_t);
+      for (Mixer& M : L.mixers) {
+        float* p[] = {M.in_bias, M.q_norm, M.k_norm, M.kv_norm, M.bias, M.sink, M.conv, M.conv_bias, M.gate_bias, M.decay, M.step_bias, M.head_norm};
+        for (float* q : p) if (q) cudaFree(q);
+        if (M.up_k_t) cudaFree(M.up_k_t);
+        if (M.gates3) cudaFree(M.gates3);
+      }
+      if (L.mixer_norm) cudaFree(L.mixer_norm);
+      if (L.mlp_norm) cudaFree(L.mlp_norm);
     }
-    float* p[] = {proj, lat_q, lat_o, att, gu, act, y, scratch};
+    float* p[] = {proj, lat_q, lat_o, att, gu, act, y, scratch, state, prep, low};
     for (float* q : p) if (q) cudaFree(q);
-    void* v[] = {x16, a16, b16};
+    void* v[] = {x16, a16, b16, freq_dev, angles, group_first};
     for (void* q : v) if (q) cudaFree(q);
   }
 };
@@ -2173,6 +2197,7 @@ int llr_session_seq_truncate(llr_session* s, size_t seq, size_t n_keep) {
   if (seq >= s->n_seq) return fail(e, LLR_ERR_INVALID, "sequence index out of range");
   if (n_keep > s->position[seq]) return fail(e, LLR_ERR_INVALID, "a sequence cannot be truncated beyond its position");
   if (n_keep == s->position[seq]) return LLR_OK;
+  if (s->dec && s->dec->state_floats > 0 && n_keep > 0) return fail(e, LLR_ERR_INVALID, "a recurrent state cannot be rewound: truncate to 0 and read the prompt again");
   DeviceGuard guard(e->device);
   if (seq == 0) {  // sequence 0 keeps its position on the device too (graph replay advances it there)
     const int p = (int)n_keep;
@@ -2374,6 +2399,13 @@ static int session_batch(llr_session* s, size_t n_groups, const uint32_t* seq_id
       (ce = cudaMemcpyAsync(s->row_seq, rseq.data(), total * sizeof(int), cudaMemcpyHostToDevice, st)) != cudaSuccess ||
       (ce = cudaMemcpyAsync(s->last_rows, last.data(), n_groups * sizeof(int), cudaMemcpyHostToDevice, st)) != cudaSuccess)
     return fail_cuda(e, ce, "batch upload");
+  if (s->dec && s->dec->state_floats > 0) {
+    std::vector<int> starts;
+    for (const auto& g : s->batch_groups) starts.push_back((int)g.first);
+    starts.push_back((int)total);
+    if ((ce = cudaMemcpyAsync(s->dec->group_first, starts.data(), starts.size() * sizeof(int), cudaMemcpyHostToDevice, st)) != cudaSuccess)
+      return fail_cuda(e, ce, "batch upload");
+  }
   const float* pending = nullptr;
   if ((ce = session_layers(s, s->ids + 1, total, RowMap{nullptr, s->row_pos, s->row_seq}, &pending)) != cudaSuccess)
     return fail_cuda(e, ce, "kernel launch");

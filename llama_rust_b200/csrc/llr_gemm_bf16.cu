@@ -9,7 +9,7 @@
 // rows (x16); results are f32, or bfloat16 for the product that follows, optionally multiplied by the sigmoid of a
 // per-head gate.
 //
-// With `glu` W stacks gate | up (2 rows rows) and the results are clamped gated units: a tile then holds as many gate rows
+// With `glu` W stacks gate | up (2 rows rows) and the results are gated units: a tile then holds as many gate rows
 // as up rows, so that a thread of the epilogue has both factors of each result.
 //
 // One CTA computes a tile of 128 activation rows x bn <= BN weight rows: the activation rows are the MMA's M dimension (one
@@ -94,11 +94,6 @@ __device__ __forceinline__ void load32(uint32_t taddr, uint32_t (&v)[32]) {
         "=r"(v[16]), "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]),
         "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
       : "r"(taddr) : "memory");
-}
-__device__ __forceinline__ float glu_of(float a, float b, const GluShape& g) {
-  a = fminf(a, g.limit);
-  b = fminf(fmaxf(b, -g.limit), g.limit);
-  return a * __fdiv_rn(1.0f, 1.0f + expf(-g.alpha * a)) * (b + g.shift);
 }
 
 template <int BN, bool GLU>
@@ -195,7 +190,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant
         float f[32];
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
-          if constexpr (GLU) f[j] = glu_of(__uint_as_float(v[j]), __uint_as_float(u[j]), a.glu);
+          if constexpr (GLU) f[j] = gated_unit(__uint_as_float(v[j]), __uint_as_float(u[j]), a.glu);
           else f[j] = a.gate ? __uint_as_float(v[j]) * gate : __uint_as_float(v[j]);
         }
         if (vec) {

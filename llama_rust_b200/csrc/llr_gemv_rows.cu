@@ -154,9 +154,7 @@ gemv_rows_glu_kernel(const uint8_t* __restrict__ W, int64_t row_bytes, int64_t c
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) { a += __shfl_xor_sync(~0u, a, o); b += __shfl_xor_sync(~0u, b, o); }
       if (lane == 0 && t < tokens) {
-        a = fminf(a, glu.limit);
-        b = fminf(fmaxf(b, -glu.limit), glu.limit);
-        Y[(int64_t)t * glu.n + row] = __fmul_rn(__fmul_rn(a, __fdiv_rn(1.0f, 1.0f + expf(-__fmul_rn(glu.alpha, a)))), __fadd_rn(b, glu.shift));
+        Y[(int64_t)t * glu.n + row] = gated_unit(a, b, glu);
       }
     }
   }

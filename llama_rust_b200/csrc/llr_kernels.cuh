@@ -305,8 +305,23 @@ cudaError_t launch_argmax_advance(const float* logits, int n, int* out_id, float
 cudaError_t launch_argmax_rows(const float* logits, int n_rows, int n, int* out_id, float* out_margin, cudaStream_t s,
                                uint64_t* launches);
 
-// Clamped gated unit: a * sigmoid(alpha * a) * (b + shift), a = min(gate, limit), b = clamp(up, -limit, limit); n results
-struct GluShape { int n; float limit, alpha, shift; };
+// Gated unit of n results.  UNIT_CLAMPED: a * sigmoid(alpha * a) * (b + shift), a = min(gate, limit), b = clamp(up, -limit,
+// limit).  UNIT_GELU: gelu(gate) * up with the tanh form of gelu.
+enum GatedUnit : int { UNIT_CLAMPED = 0, UNIT_GELU = 1 };
+struct GluShape { int n; float limit, alpha, shift; int unit; };
+#ifdef __CUDACC__
+// 0.5 z (1 + tanh(w)) = z sigmoid(2 w), w = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) {
+  const float w2 = __fmul_rn(1.5957691216057308f, __fmul_rn(z, fmaf(0.044715f, __fmul_rn(z, z), 1.0f)));
+  return __fdiv_rn(z, 1.0f + expf(-w2));
+}
+__device__ __forceinline__ float gated_unit(float a, float b, const GluShape& g) {
+  if (g.unit == UNIT_GELU) return __fmul_rn(gelu_tanh(a), b);
+  a = fminf(a, g.limit);
+  b = fminf(fmaxf(b, -g.limit), g.limit);
+  return __fmul_rn(__fmul_rn(a, __fdiv_rn(1.0f, 1.0f + expf(-__fmul_rn(g.alpha, a)))), __fadd_rn(b, g.shift));
+}
+#endif
 // ---- products with bfloat16 weights for many rows (llr_gemm_bf16.cu): tcgen05, bfloat16 activations, f32 accumulation ----
 // y[t * y_ld + z * rows + r] = sum_c W[z * rows + r][c] x[t][z * xk + c] for z < batch (a product per head), times
 // sigmoid(gate[t * gate_ld + z]) when gate is set.  Results as f32 (y), as bfloat16 (y16), or both.  With slices > 1
@@ -320,7 +335,7 @@ struct Bf16Product {
   const float* gate;
   int64_t y_ld, gate_ld, slice_stride;
   int tokens, rows, cols, batch, xk, slices;
-  const GluShape* glu;  // W stacks gate | up, 2 rows rows: the results are clamped gated units (batch 1)
+  const GluShape* glu;  // W stacks gate | up, 2 rows rows: the results are gated units (batch 1)
 };
 bool gemm_bf16_supported(const void* w, int64_t rows, int64_t cols);
 int gemm_bf16_slices(int tokens, int rows, int cols);
@@ -340,21 +355,38 @@ struct LayerKv {
 };
 // What a row attends to and how it scores: n_head query heads over n_kv key/value heads (n_head / n_kv share one), the
 // last `window` positions (0: all) and the first keep_first; score = (q . k) * scale + bias[h][min(distance, bias_len - 1)].
+// sink[h] (may be null) is one more score that has no value: exp(sink) stands in the denominator.
 struct SpanShape {
   int n_head, n_kv, dk, dv, window, keep_first, n_ctx;
   float scale;
   const float* bias;  // [n_head][bias_len], or null
   int bias_len;
+  const float* sink;  // [n_head], or null
+};
+// Rotation of a head's first dims values, pairs (i, i + dims / 2): row t's cosines and sines are the dims / 2 entries from
+// cs + t * ld on.  dims 0: none.
+struct RotRows {
+  const float2* cs;
+  int ld, dims;
+};
+// Every distinct rotation of a model, end to end: cs[t * n + i] = (cos, sin)(position of t * freq[i])
+struct RotTable {
+  const double* freq;
+  float2* cs;
+  int n;
 };
 // x[t] = table[ids[t]] * scale + pos_table[position of t]; table and pos_table (may be null) are bfloat16 rows of n.
-// x16 (may be null): the same as bfloat16.
+// x16 (may be null): the same as bfloat16.  The rows' rotation angles are taken here too, once for all layers.
 cudaError_t launch_embed(const void* table, const void* pos_table, const int* ids, const RowMap& rows, float scale, float* x,
-                         void* x16, int tokens, int n, cudaStream_t s, uint64_t* launches);
+                         void* x16, int tokens, int n, const RotTable& rot, cudaStream_t s, uint64_t* launches);
 // q | k | v of a stacked projection (row t at proj + t * ld): bias added; q and k divided by the root mean square of the
-// WHOLE projection and weighted, where norms are given; k and v into the cache, q left in place.
+// WHOLE projection and weighted, where norms are given, then rotated; k and v into the cache, q left in place.
+// `also` (heads 0: none): heads of a mixer beside this one in the same rows, rotated in place.
 struct QkvShape { int n_head, n_kv, dk, dv; float eps; };
-cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh,
-                             const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
+struct RotHeads { float* x; int heads, dim; RotRows rot; };  // heads * dim values at x + t * ld
+cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh, const RotRows& rot,
+                             const RotHeads& also, const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
+cudaError_t launch_rotate_heads(const RotHeads& h, int ld, int tokens, cudaStream_t s, uint64_t* launches);
 // One latent per row (n floats at proj + t * ld): normed, weighted, into the cache.  q16 (may be null): the nq floats at
 // q + t * ld as bfloat16 rows of nq.
 cudaError_t launch_latent_store(const float* proj, int ld, const float* w, int n, float eps, const LayerKv& kv, const RowMap& rows,
@@ -369,8 +401,7 @@ cudaError_t launch_head_product_t(const void* w, int heads, int rows, int cols, 
 cudaError_t launch_head_product(const void* w, int heads, int rows, int cols, const float* x, int64_t x_ld, float* y, const float* gate,
                                 int64_t gate_ld, int tokens, cudaStream_t s, uint64_t* launches);
 cudaError_t launch_head_transpose(const void* w, int heads, int rows, int cols, void* out, cudaStream_t s, uint64_t* launches);
-// Attention over the visible keys.  q: row t at q + t * q_ld.  Result rows of n_head * dv, f32 (out) and/or bfloat16 (out16);
-// gate (may be null): element gate, result times sigmoid(gate[t * gate_ld + h * dv + i]).
+// Attention over the visible keys.  q: row t at q + t * q_ld.  Results go where SpanOut says.
 // one_sequence: the rows are one sequence at consecutive positions; with tensor_cores such rows may run as binary16 MMAs.
 // A single decode token whose projection the attention kernel takes in itself (null proj: it is in the cache already):
 // the row's stacked q | k | v with launch_qkv_store's arguments, or (latent) its latent with the weights in k_norm.
@@ -378,17 +409,119 @@ struct NewToken {
   const float *proj = nullptr, *bias = nullptr, *q_norm = nullptr, *k_norm = nullptr;
   float eps = 0.f;
   bool latent = false;
+  RotRows rot{};
+};
+// Row t's results: n_head * dv values from t * ld on, f32 (out) and/or bfloat16 (out16), times `scale` and, with a gate,
+// times sigmoid(gate[t * gate_ld + h * dv + i]) or (head_gate) sigmoid(gate[t * gate_ld + h]).
+struct SpanOut {
+  float* out;
+  void* out16;
+  int64_t ld;
+  const float* gate;
+  int64_t gate_ld;
+  bool head_gate;
+  float scale;
 };
 size_t span_scratch_floats(const SpanShape& sh, int max_rows);
 bool span_supported(const SpanShape& sh);
 cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape& sh, const LayerKv& kv, const RowMap& rows, int t0, int tokens,
-                                  float* out, void* out16, const float* gate, int64_t gate_ld, float* scratch, bool tensor_cores,
-                                  bool one_sequence, const NewToken* nt, cudaStream_t s, uint64_t* launches);
+                                  const SpanOut& out, float* scratch, bool tensor_cores, bool one_sequence, const NewToken* nt, cudaStream_t s,
+                                  uint64_t* launches);
 // x[t] += y[t] / rms(y[t]) * w, y given as `slices` partial sums `slice_stride` floats apart; x16 (may be null): the new x
 cudaError_t launch_norm_add(float* x, const float* y, int slices, int64_t slice_stride, const float* w, float eps, void* x16, int tokens, int n,
                             cudaStream_t s, uint64_t* launches);
-// the clamped gated unit of a stacked product: row t of gu is gate | up, n each
-cudaError_t launch_clamped_glu(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches);
+// x[t] += y[t] (slices 0: nothing to add), then, with w, h[t] = x[t] / rms(x[t]) * w as f32 (h) and / or bfloat16 (h16)
+cudaError_t launch_add_norm(float* x, const float* y, int slices, int64_t slice_stride, const float* w, float eps, float* h, void* h16, int tokens,
+                            int n, cudaStream_t s, uint64_t* launches);
+// the gated unit of a stacked product: row t of gu is gate | up, n each
+cudaError_t launch_gated_unit(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches);
+
+// ---- recurrent mixers (llr_recurrent.cu): a state per sequence instead of cached positions ----
+// The groups of a batch: group i has the rows [first[i], first[i + 1]) of one sequence at consecutive positions; null: one
+// group of all rows.  A group whose first row stands at position 0 starts from a state of zeros, whatever memory holds.
+struct RowGroups {
+  const int* first;
+  int n, longest;
+};
+// A mixer's state of sequence q lies at state + q * stride.
+struct StateView {
+  float* state;
+  int64_t stride;
+};
+// Short causal convolution per channel over the rows of a sequence: w [channels][taps], the last tap weighs the row itself.
+// bias is added to the inputs, out_bias to the results (both may be null); tail: the state's last taps - 1 inputs
+// [taps - 1][channels].
+struct ConvShape {
+  const float *w, *bias, *out_bias;
+  int channels, taps;
+  StateView tail;
+};
+// What follows a head's result o (vdim values): o / rms(o) (times weight), times sigmoid or silu of its gate row, times
+// scale; f32 and / or bfloat16 rows at t * ld.
+struct HeadOut {
+  const float *weight, *gate;
+  int64_t gate_ld;
+  bool silu;
+  float eps, scale;
+  float* out;
+  void* out16;
+  int64_t ld;
+};
+// Matrix states S [dim][vdim] per head, one column of S per eight lanes, f32.  Row t: q, k (n_kv heads of dim, head h reads
+// h / (n_head / n_kv)) and v (n_head of vdim) at + t * ld.
+//   retention (g null):  S = decay[h] S + (k scale) v^T, o = S^T q; a single row may come unrotated (rot)
+//   delta rule:          S = diag(g) S, u = beta (v - S^T k), S += k u^T, o = S^T q; g [n_head][dim], beta [n_head],
+//                        kq [n_kv] = k . q at + t * ld too
+struct MatrixScan {
+  const float *q, *k, *v, *g, *beta, *kq, *decay;
+  int64_t ld, v_ld;
+  int n_head, n_kv, dim, vdim;
+  float k_scale;
+  RotRows rot;
+  StateView state;
+  // delta rule: the convolution's inputs, whose last rows replace the state's tail behind the scan
+  const float* conv_in;
+  int64_t conv_ld;
+  ConvShape conv;
+};
+bool matrix_scan_supported(int dim, int vdim);
+// o_scratch: [tokens][n_head * vdim] floats
+cudaError_t launch_matrix_scan(const MatrixScan& m, const HeadOut& out, const RowGroups& groups, const RowMap& rows, int tokens, float* o_scratch,
+                               cudaStream_t s, uint64_t* launches);
+// Inputs of the delta rule from a row of projections q | k | v: convolution, silu, q and k as unit vectors (x / sqrt(sum x^2 +
+// unit_eps)), q times q_scale; g = exp(-rate[h] softplus(a + step_bias)), beta = sigmoid(b).
+// Row t of prep (prep_ld floats): q | k | v | g | beta | k . q.
+struct DeltaShape {
+  int n_head, n_kv, dim, vdim;
+  float q_scale, unit_eps;
+  const float *rate, *step_bias;  // [n_head], [n_head * dim]
+};
+int delta_prep_floats(const DeltaShape& d);
+bool delta_supported(const DeltaShape& d);
+cudaError_t launch_delta_prepare(const float* proj, int64_t ld, const float* a, const float* b, const DeltaShape& d, const ConvShape& conv, float* prep,
+                                 const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
+// u[t] = convolution of the rows at x + t * ld.  u16 (may be null): u as three bfloat16 parts whose sum it is, per block of
+// `block` channels: [channels / block][3][block].
+cudaError_t launch_conv_rows(const float* x, int64_t ld, const ConvShape& conv, float* u, void* u16, int block, const RowMap& rows, int tokens,
+                             cudaStream_t s, uint64_t* launches);
+// Real-gated linear recurrence per channel: r, i = sigmoid(gates + gate_bias) (row t of gates: per block r | i), log a =
+// -rate r, S = a S + sqrt(1 - a^2) i u; result S gelu(y + y_bias).
+struct GatedScan {
+  const float *gates, *gate_bias, *u, *rate, *y, *y_bias;
+  int64_t y_ld;
+  int width, block;
+  StateView state;
+  const float* conv_in;  // as in MatrixScan
+  int64_t conv_ld;
+  ConvShape conv;
+  float* out;
+  void* out16;
+  int64_t ld;
+  float scale;
+};
+cudaError_t launch_gated_scan(const GatedScan& g, const RowGroups& groups, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
+// W with every block of `cols` columns three times in a row, for products with u16 (once per session)
+cudaError_t launch_triple_columns(const void* w, int64_t rows, int cols, void* out, cudaStream_t s, uint64_t* launches);
 
 // *flag_dev = 1 when the two device byte ranges differ (both 16-byte aligned), else 0
 cudaError_t launch_bytes_differ(const void* a, const void* b, size_t n, int* flag_dev, cudaStream_t stream, uint64_t* launches);

@@ -3,8 +3,10 @@
 // per head and distance bucket, a sliding window that keeps the first tokens, and an element-wise output gate, or
 // (b) latent attention: one normed latent vector per position is cached and serves every head; a head's query is taken
 // into the latent space (q' = W_uk^T q, so that q . (W_uk c) = q' . c) and its result out of it (W_uv (sum p c)).
-// Then the norm on a sublayer's output with its residual add, the clamped gated unit, and the embedding with learned
-// positions.  Sizes and constants are arguments; a mechanism that is absent is a null pointer or a zero.
+// Heads may be rotated by their position, and a softmax may have a sink: a score without a key.
+// Then the norms of the residual stream -- on a sublayer's output before its add, or on its input behind the add of the one
+// before --, the gated unit, and the embedding with learned positions.  Sizes and constants are arguments; a mechanism that
+// is absent is a null pointer or a zero.
 //
 // Scores, softmax, norms, sigmoids and the residual stream are f32 throughout.
 #include <cuda_bf16.h>
@@ -34,9 +36,18 @@ __device__ __forceinline__ float4 widen4(uint2 u) {
 // ---- embedding ------------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256)
 embed_kernel(const uint16_t* __restrict__ table, const uint16_t* __restrict__ pos_table, const int* __restrict__ ids, RowMap rows, float scale,
-             float* __restrict__ x, __nv_bfloat16* __restrict__ x16, int n) {
+             float* __restrict__ x, __nv_bfloat16* __restrict__ x16, int n, RotTable rot) {
   pdl_enter();
   const int t = blockIdx.x;
+  if (rot.n > 0) {  // angles reduced in double precision: far positions keep every bit their float cosine can hold
+    const double pos = (double)row_position(rows, t);
+    for (int i = threadIdx.x; i < rot.n; i += blockDim.x) {
+      const double turns = pos * rot.freq[i] * 0.15915494309189535;  // 1 / (2 pi)
+      float sn, cs;
+      sincospif((float)(2.0 * (turns - rint(turns))), &sn, &cs);
+      rot.cs[(int64_t)t * rot.n + i] = make_float2(cs, sn);
+    }
+  }
   const uint16_t* e = table + (int64_t)ids[t] * n;
   const uint16_t* p = pos_table ? pos_table + (int64_t)row_position(rows, t) * n : nullptr;
   for (int i = 4 * threadIdx.x; i < n; i += 4 * blockDim.x) {  // n is a multiple of four
@@ -109,10 +120,46 @@ __device__ __forceinline__ QkvRow qkv_row(const float* p, int ld, const float* b
   return r;
 }
 
+// Value i of a run of heads of d values whose values before the rotation are f(i); cs: the row's cosines and sines
+template <typename F>
+__device__ __forceinline__ float rotated(const F& f, int i, int d, const float2* cs, int dims) {
+  const int c = i % d, half = dims / 2;
+  const float v = f(i);
+  if (c >= dims) return v;
+  const float2 a = cs[c < half ? c : c - half];
+  return c < half ? fmaf(v, a.x, -__fmul_rn(f(i + half), a.y)) : fmaf(v, a.x, __fmul_rn(f(i - half), a.y));
+}
+// The same for all n values in place: a pair belongs to one thread.  f(i) reads x[i].
+template <typename F>
+__device__ __forceinline__ void rotate_in_place(const F& f, float* x, int n, int d, const float2* cs, int dims) {
+  const int half = dims / 2, own = d - half;  // a head's pairs, then what passes unchanged
+  for (int j = threadIdx.x; j < n / d * own; j += blockDim.x) {
+    const int c = j % own, i = j / own * d + (c < half ? c : c + half);
+    const float u = f(i);
+    if (c < half) {
+      const float v = f(i + half);
+      const float2 a = cs[c];
+      x[i] = fmaf(u, a.x, -__fmul_rn(v, a.y));
+      x[i + half] = fmaf(v, a.x, __fmul_rn(u, a.y));
+    } else {
+      x[i] = u;
+    }
+  }
+}
+__device__ __forceinline__ void rotate_heads(const RotHeads& h, int64_t ld, int t) {
+  float* x = h.x + (int64_t)t * ld;
+  rotate_in_place([&](int i) { return x[i]; }, x, h.heads * h.dim, h.dim, h.rot.cs + (int64_t)t * h.rot.ld, h.rot.dims);
+}
+__global__ void __launch_bounds__(256)
+rotate_heads_kernel(RotHeads h, int ld) {
+  pdl_enter();
+  rotate_heads(h, ld, blockIdx.x);
+}
+
 // one block per row
 __global__ void __launch_bounds__(PROJ_THREADS)
 qkv_store_kernel(float* proj, int ld, const float* __restrict__ bias, const float* __restrict__ q_norm,
-                 const float* __restrict__ k_norm, QkvShape sh, LayerKv kv, RowMap rows) {
+                 const float* __restrict__ k_norm, QkvShape sh, RotRows rot, RotHeads also, LayerKv kv, RowMap rows) {
   pdl_enter();
   __shared__ float red[2][32];
   const int t = blockIdx.x, nk = sh.n_kv * sh.dk, nv = sh.n_kv * sh.dv;
@@ -122,9 +169,16 @@ qkv_store_kernel(float* proj, int ld, const float* __restrict__ bias, const floa
   // the page and the place in it once; heads lie block_tokens vectors apart
   float* k0 = kv.k + slot_of(kv, seq, pos, kv.k_block, 0, sh.dk);
   float* v0 = kv.v + slot_of(kv, seq, pos, kv.v_block, 0, sh.dv);
-  for (int i = threadIdx.x; i < nk; i += PROJ_THREADS) k0[(int64_t)(i / sh.dk) * kv.block_tokens * sh.dk + i % sh.dk] = r.k(i);
+  if (also.heads > 0) rotate_heads(also, ld, t);
+  const float2* cs = rot.dims > 0 ? rot.cs + (int64_t)t * rot.ld : nullptr;
+  const auto qf = [&](int i) { return r.q(i); };
+  const auto kf = [&](int i) { return r.k(i); };
+  for (int i = threadIdx.x; i < nk; i += PROJ_THREADS)
+    k0[(int64_t)(i / sh.dk) * kv.block_tokens * sh.dk + i % sh.dk] = cs ? rotated(kf, i, sh.dk, cs, rot.dims) : r.k(i);
   for (int i = threadIdx.x; i < nv; i += PROJ_THREADS) v0[(int64_t)(i / sh.dv) * kv.block_tokens * sh.dv + i % sh.dv] = r.v(i);
-  if (bias || q_norm) {
+  if (cs) {
+    rotate_in_place(qf, p, r.nq, sh.dk, cs, rot.dims);
+  } else if (bias || q_norm) {
     for (int i0 = threadIdx.x; i0 < r.nq; i0 += 4 * PROJ_THREADS) {  // four values in flight; each is read and written by one thread
       float u[4];
 #pragma unroll
@@ -226,7 +280,7 @@ head_product_kernel(const uint16_t* __restrict__ w, int heads, int rows, int col
   float acc[TT];
 #pragma unroll
   for (int j = 0; j < TT; ++j) acc[j] = 0.f;
-  if ((cols & 3) == 0 && (x_ld & 3) == 0) {
+  if ((cols & 3) == 0 && (x_ld & 3) == 0 && ((uintptr_t)x & 15) == 0) {
 #pragma unroll 4
     for (int c = 4 * lane; c < cols; c += 128) {
       const uint2 u = *(const uint2*)(wr + c);
@@ -295,6 +349,10 @@ struct KvSpan {
   }
 };
 
+// Keys of a slice for a row that sees n of them: 32 slices once there are enough keys, so that a short sequence in a long
+// context still spreads over the SMs.  Never more than the chunk the launch is sized for.
+__device__ __forceinline__ int span_step(int n) { return max(32, (n + 31) / 32); }
+
 // Query heads of a kv head that share a block: eight, four where a head's query and value rows are long.
 inline __host__ __device__ int span_heads(const SpanShape& sh) { return sh.dk + sh.dv > 512 ? ATT_MAX_GQA / 2 : ATT_MAX_GQA; }
 
@@ -316,7 +374,7 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
   const int t = t0 + blockIdx.z, split = blockIdx.y, n_split = (int)gridDim.y, h0 = head * gq + g0;
   const int pos = row_position(rows, t);
   const Span span = span_of(pos, sh.window, sh.keep_first);
-  const int s0 = split * chunk, s1 = min(span.n, s0 + chunk);
+  const int step = span_step(span.n), s0 = split * step, s1 = min(span.n, s0 + step);
   if (s0 >= span.n) return;
   float* sq = sm;
   float* sc = sq + heads * sh.dk;
@@ -327,11 +385,16 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
   if (nt.proj && !nt.latent) {
     const QkvShape qs{sh.n_head, sh.n_kv, sh.dk, sh.dv, nt.eps};
     const QkvRow r = qkv_row(nt.proj, (int)q_ld, nt.bias, nt.q_norm, nt.k_norm, qs, red);
-    for (int i = threadIdx.x; i < heads * sh.dk; i += ATT_THREADS) sq[i] = r.q(h0 * sh.dk + i);
+    const float2* cs = nt.rot.dims > 0 ? nt.rot.cs + (int64_t)t * nt.rot.ld : nullptr;
+    const auto qf = [&](int i) { return r.q(i); };
+    const auto kf = [&](int i) { return r.k(i); };
+    for (int i = threadIdx.x; i < heads * sh.dk; i += ATT_THREADS)
+      sq[i] = cs ? rotated(qf, h0 * sh.dk + i, sh.dk, cs, nt.rot.dims) : r.q(h0 * sh.dk + i);
     if (s1 == span.n) {
       float* k = kv.k + slot_of(kv, row_sequence(rows, t), pos, kv.k_block, head, sh.dk);
       float* v = kv.v + slot_of(kv, row_sequence(rows, t), pos, kv.v_block, head, sh.dv);
-      for (int i = threadIdx.x; i < sh.dk; i += ATT_THREADS) k[i] = r.k(head * sh.dk + i);
+      for (int i = threadIdx.x; i < sh.dk; i += ATT_THREADS)
+        k[i] = cs ? rotated(kf, head * sh.dk + i, sh.dk, cs, nt.rot.dims) : r.k(head * sh.dk + i);
       for (int i = threadIdx.x; i < sh.dv; i += ATT_THREADS) v[i] = r.v(head * sh.dv + i);
     }
   } else {
@@ -344,21 +407,22 @@ span_partial_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, Lay
   attend_slice<MAX_VALUE>(KvSpan{kv, sh, smw, span, s0, head, pos, h0}, sq, sc, rec, s0, s1, chunk, sh.dk, sh.dv, heads);
 }
 
-// grid (query head, row, 128 dimensions): merges a head's slices (at most 32) and applies the element gate
+// grid (query head, row, 128 dimensions): merges a head's slices (at most 32) and the sink, applies the gate
 __global__ void __launch_bounds__(128)
-span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, int t0, int chunk, int n_split, float* __restrict__ out,
-                    __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate, int64_t gate_ld) {
+span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, int t0, int n_split, SpanOut so) {
   pdl_enter();
   const int lane = threadIdx.x & 31, h = blockIdx.x, t = t0 + blockIdx.y;
   const int gq = sh.n_head / sh.n_kv, per = span_heads(sh), groups = (gq + per - 1) / per;
   const int bx = (h / gq) * groups + (h % gq) / per, g = (h % gq) % per;
-  const int used = (span_of(row_position(rows, t), sh.window, sh.keep_first).n + chunk - 1) / chunk;
+  const int seen = span_of(row_position(rows, t), sh.window, sh.keep_first).n, step = span_step(seen), used = (seen + step - 1) / step;
   const int64_t stride = (int64_t)per * (sh.dv + 2);
   const float* base = part + ((int64_t)blockIdx.y * sh.n_kv * groups + bx) * n_split * stride + g * (sh.dv + 2);
   const float ms = lane < used ? base[lane * stride + sh.dv] : -CUDART_INF_F;
-  const float m = warp_max(ms);
+  float m = warp_max(ms);
+  if (sh.sink) m = fmaxf(m, sh.sink[h]);
   const float e = lane < used ? expf(ms - m) : 0.f;
-  const float l = warp_sum(lane < used ? base[lane * stride + sh.dv + 1] * e : 0.f);
+  float l = warp_sum(lane < used ? base[lane * stride + sh.dv + 1] * e : 0.f);
+  if (sh.sink) l = __fadd_rn(l, expf(sh.sink[h] - m));
   const int i = blockIdx.z * 128 + threadIdx.x;
   const bool live = i < sh.dv;
   float acc = 0.f;
@@ -372,9 +436,10 @@ span_combine_kernel(const float* __restrict__ part, SpanShape sh, RowMap rows, i
   if (live) {
     float r = __fdiv_rn(acc, l);
     const int64_t o = (int64_t)h * sh.dv + i;
-    if (gate) r = __fmul_rn(r, sigmoid(gate[(int64_t)t * gate_ld + o]));
-    if (out) out[(int64_t)t * sh.n_head * sh.dv + o] = r;
-    if (out16) out16[(int64_t)t * sh.n_head * sh.dv + o] = __float2bfloat16_rn(r);
+    if (so.gate) r = __fmul_rn(r, sigmoid(so.gate[(int64_t)t * so.gate_ld + (so.head_gate ? h : o)]));
+    r = __fmul_rn(r, so.scale);
+    if (so.out) so.out[(int64_t)t * so.ld + o] = r;
+    if (so.out16) ((__nv_bfloat16*)so.out16)[(int64_t)t * so.ld + o] = __float2bfloat16_rn(r);
   }
 }
 
@@ -471,8 +536,7 @@ span_gather_kernel(SpanShape sh, LayerKv kv, RowMap rows, int t0, int tokens, in
 template <int ND, int NS>
 __global__ void __launch_bounds__(128 * NS)
 span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, const __half* __restrict__ k16, const __half* __restrict__ v16, bool shared_kv,
-                RowMap rows, int t0, int tokens, float* __restrict__ out, __nv_bfloat16* __restrict__ out16, const float* __restrict__ gate,
-                int64_t gate_ld) {
+                RowMap rows, int t0, int tokens, SpanOut so) {
   pdl_enter();
   constexpr int THR = 128 * NS, NT = CH / 8 / NS;  // score tiles of eight keys per warp
   static_assert(NT % 2 == 0, "keys are loaded sixteen at a time");
@@ -529,6 +593,11 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, const _
   const float far0 = b0 ? b0[sh.bias_len - 1] * LOG2E : 0.f, far1 = b1 ? b1[sh.bias_len - 1] * LOG2E : 0.f;
   const float f0 = s_scale[r0] * LOG2E, f1 = s_scale[r1] * LOG2E;
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
+  if (sh.sink) {  // the sink is the first score: the maximum starts there, and one thread of a row's counts it
+    m0 = sh.sink[head * gq + min(pair0 + r0, pairs - 1) % gq] * LOG2E;
+    m1 = sh.sink[head * gq + min(pair0 + r1, pairs - 1) % gq] * LOG2E;
+    l0 = l1 = t4 == 0 && ns == 0 ? 1.f : 0.f;
+  }
   float o[ND][4];
 #pragma unroll
   for (int nd = 0; nd < ND; ++nd)
@@ -671,21 +740,22 @@ span_mma_kernel(const float* __restrict__ q, int64_t q_ld, SpanShape sh, const _
     const int p = pair0 + (half ? r1 : r0);
     if (p >= pairs) continue;
     const int t = t0 + p / gq, h = head * gq + p % gq;
-    const float inv = __fdiv_rn(1.0f, half ? l1 : l0);
+    float inv = __fdiv_rn(1.0f, half ? l1 : l0) * so.scale;
+    if (so.gate && so.head_gate) inv *= sigmoid(so.gate[(int64_t)t * so.gate_ld + h]);
     const int64_t base = (int64_t)h * sh.dv;
 #pragma unroll
     for (int nd = 0; nd < ND; ++nd) {
       const int d = ns * 8 * ND + 8 * nd + 2 * t4;
       if (d >= sh.dv) continue;
       float2 v = make_float2(o[nd][2 * half] * inv, o[nd][2 * half + 1] * inv);
-      if (gate) {
-        const float2 gg = *(const float2*)(gate + (int64_t)t * gate_ld + base + d);
+      if (so.gate && !so.head_gate) {
+        const float2 gg = *(const float2*)(so.gate + (int64_t)t * so.gate_ld + base + d);
         v.x *= sigmoid(gg.x);
         v.y *= sigmoid(gg.y);
       }
-      const int64_t at = (int64_t)t * sh.n_head * sh.dv + base + d;
-      if (out) *(float2*)(out + at) = v;
-      if (out16) *(__nv_bfloat162*)(out16 + at) = __floats2bfloat162_rn(v.x, v.y);
+      const int64_t at = (int64_t)t * so.ld + base + d;
+      if (so.out) *(float2*)(so.out + at) = v;
+      if (so.out16) *(__nv_bfloat162*)((__nv_bfloat16*)so.out16 + at) = __floats2bfloat162_rn(v.x, v.y);
     }
   }
 }
@@ -748,14 +818,62 @@ norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, int slices, 
   }
 }
 
-// ---- clamped gated unit -------------------------------------------------------------------------------------------
-__device__ __forceinline__ float clamped_glu(float a, float b, const GluShape& sh) {
-  a = fminf(a, sh.limit);
-  b = fminf(fmaxf(b, -sh.limit), sh.limit);
-  return __fmul_rn(__fmul_rn(a, sigmoid(__fmul_rn(sh.alpha, a))), __fadd_rn(b, sh.shift));
+// ---- residual add, norm of the sum: what a sublayer reads ------------------------------------------------------------
+__global__ void __launch_bounds__(NORM_ADD_THREADS)
+add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, int slices, int64_t slice_stride, const float* __restrict__ w, float eps,
+                float* __restrict__ h, __nv_bfloat16* __restrict__ h16, int n) {
+  pdl_enter();
+  __shared__ float sh[32];
+  const int64_t row = (int64_t)blockIdx.x * n;
+  const bool in_regs = n <= 4 * NORM_ADD_THREADS * NORM_ADD_KEEP;  // n is a multiple of four
+  auto fresh = [&](int i) {  // the new residual values
+    float4 v = *(const float4*)(x + row + i);
+    if (slices > 0) {
+      float4 a = *(const float4*)(y + row + i);
+      for (int s = 1; s < slices; ++s) {
+        const float4 u = *(const float4*)(y + s * slice_stride + row + i);
+        a.x += u.x; a.y += u.y; a.z += u.z; a.w += u.w;
+      }
+      v = make_float4(__fadd_rn(v.x, a.x), __fadd_rn(v.y, a.y), __fadd_rn(v.z, a.z), __fadd_rn(v.w, a.w));
+      *(float4*)(x + row + i) = v;
+    }
+    return v;
+  };
+  float4 keep[NORM_ADD_KEEP];
+  float ss = 0.f;
+  auto square = [&](float4 v) { ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); };
+  if (in_regs) {
+#pragma unroll
+    for (int k = 0; k < NORM_ADD_KEEP; ++k) {
+      const int i = 4 * (threadIdx.x + k * NORM_ADD_THREADS);
+      if (i < n) { keep[k] = fresh(i); square(keep[k]); }
+    }
+  } else {
+    for (int i = 4 * threadIdx.x; i < n; i += 4 * NORM_ADD_THREADS) square(fresh(i));
+  }
+  if (!w) return;
+  const float inv = inv_rms(block_sum(ss, sh), n, eps);
+  auto put = [&](int i, float4 v) {
+    const float4 ww = *(const float4*)(w + i);
+    v = make_float4(__fmul_rn(__fmul_rn(v.x, inv), ww.x), __fmul_rn(__fmul_rn(v.y, inv), ww.y), __fmul_rn(__fmul_rn(v.z, inv), ww.z),
+                    __fmul_rn(__fmul_rn(v.w, inv), ww.w));
+    if (h) *(float4*)(h + row + i) = v;
+    if (h16) *(uint2*)(h16 + row + i) = pack4_bf16(v);
+  };
+  if (in_regs) {
+#pragma unroll
+    for (int k = 0; k < NORM_ADD_KEEP; ++k) {
+      const int i = 4 * (threadIdx.x + k * NORM_ADD_THREADS);
+      if (i < n) put(i, keep[k]);
+    }
+  } else {
+    for (int i = 4 * threadIdx.x; i < n; i += 4 * NORM_ADD_THREADS) put(i, *(const float4*)(x + row + i));  // this thread's own
+  }
 }
+
+// ---- gated unit ----------------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256)
-clamped_glu_kernel(const float* __restrict__ gu, GluShape sh, float* __restrict__ out, __nv_bfloat16* __restrict__ out16, int tokens) {
+gated_unit_kernel(const float* __restrict__ gu, GluShape sh, float* __restrict__ out, __nv_bfloat16* __restrict__ out16, int tokens) {
   pdl_enter();
   const int64_t step = (int64_t)gridDim.x * blockDim.x, first = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (sh.n % 4 == 0) {
@@ -763,7 +881,7 @@ clamped_glu_kernel(const float* __restrict__ gu, GluShape sh, float* __restrict_
     for (int64_t i = first; i < (int64_t)tokens * n4; i += step) {
       const int64_t t = i / n4, c = 4 * (i % n4);
       const float4 a = *(const float4*)(gu + t * 2 * sh.n + c), b = *(const float4*)(gu + t * 2 * sh.n + sh.n + c);
-      const float4 r = make_float4(clamped_glu(a.x, b.x, sh), clamped_glu(a.y, b.y, sh), clamped_glu(a.z, b.z, sh), clamped_glu(a.w, b.w, sh));
+      const float4 r = make_float4(gated_unit(a.x, b.x, sh), gated_unit(a.y, b.y, sh), gated_unit(a.z, b.z, sh), gated_unit(a.w, b.w, sh));
       if (out) *(float4*)(out + t * sh.n + c) = r;
       if (out16) *(uint2*)(out16 + t * sh.n + c) = pack4_bf16(r);
     }
@@ -771,7 +889,7 @@ clamped_glu_kernel(const float* __restrict__ gu, GluShape sh, float* __restrict_
   }
   for (int64_t i = first; i < (int64_t)tokens * sh.n; i += step) {
     const int64_t t = i / sh.n, c = i % sh.n;
-    const float r = clamped_glu(gu[t * 2 * sh.n + c], gu[t * 2 * sh.n + sh.n + c], sh);
+    const float r = gated_unit(gu[t * 2 * sh.n + c], gu[t * 2 * sh.n + sh.n + c], sh);
     if (out) out[i] = r;
     if (out16) out16[i] = __float2bfloat16_rn(r);
   }
@@ -801,8 +919,7 @@ int span_group_keys(const SpanShape& sh, int rows) {
 }
 constexpr size_t MMA_SMEM_LIMIT = 222 * 1024;
 
-typedef void (*MmaKernel)(const float*, int64_t, SpanShape, const __half*, const __half*, bool, RowMap, int, int, float*, __nv_bfloat16*, const float*,
-                          int64_t);
+typedef void (*MmaKernel)(const float*, int64_t, SpanShape, const __half*, const __half*, bool, RowMap, int, int, SpanOut);
 // the smallest instantiation that covers the value dimensions
 MmaKernel mma_kernel(int dv, int* nd, int* ns) {
 #define LLR_SPAN(N, S) if (dv <= 8 * N * S) { *nd = N; *ns = S; return span_mma_kernel<N, S>; }
@@ -814,18 +931,24 @@ MmaKernel mma_kernel(int dv, int* nd, int* ns) {
 }  // namespace
 
 cudaError_t launch_embed(const void* table, const void* pos_table, const int* ids, const RowMap& rows, float scale, float* x, void* x16,
-                         int tokens, int n, cudaStream_t s, uint64_t* launches) {
+                         int tokens, int n, const RotTable& rot, cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
   return launch_walk(embed_kernel, dim3(tokens), dim3(256), 0, s, (const uint16_t*)table, (const uint16_t*)pos_table, ids, rows, scale, x,
-                     (__nv_bfloat16*)x16, n);
+                     (__nv_bfloat16*)x16, n, rot);
 }
 
-cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh,
-                             const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches) {
+cudaError_t launch_qkv_store(float* proj, int ld, const float* bias, const float* q_norm, const float* k_norm, const QkvShape& sh, const RotRows& rot,
+                             const RotHeads& also, const LayerKv& kv, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
-  return launch_walk(qkv_store_kernel, dim3(tokens), dim3(PROJ_THREADS), 0, s, proj, ld, bias, q_norm, k_norm, sh, kv, rows);
+  return launch_walk(qkv_store_kernel, dim3(tokens), dim3(PROJ_THREADS), 0, s, proj, ld, bias, q_norm, k_norm, sh, rot, also, kv, rows);
+}
+
+cudaError_t launch_rotate_heads(const RotHeads& h, int ld, int tokens, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0 || h.heads <= 0 || h.rot.dims <= 0) return cudaSuccess;
+  if (launches) ++*launches;
+  return launch_walk(rotate_heads_kernel, dim3(tokens), dim3(256), 0, s, h, ld);
 }
 
 cudaError_t launch_latent_store(const float* proj, int ld, const float* w, int n, float eps, const LayerKv& kv, const RowMap& rows, int tokens,
@@ -884,12 +1007,13 @@ size_t span_scratch_floats(const SpanShape& sh, int max_rows) {
 }
 
 cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape& sh, const LayerKv& kv, const RowMap& rows, int t0, int tokens,
-                                  float* out, void* out16, const float* gate, int64_t gate_ld, float* scratch, bool tensor_cores, bool one_sequence,
-                                  const NewToken* nt, cudaStream_t s, uint64_t* launches) {
+                                  const SpanOut& out, float* scratch, bool tensor_cores, bool one_sequence, const NewToken* nt, cudaStream_t s,
+                                  uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (!span_supported(sh)) return cudaErrorInvalidValue;
   const int gq = sh.n_head / sh.n_kv;
-  if (tensor_cores && one_sequence && sh.dk % 8 == 0 && sh.dv % 8 == 0 && q_ld % 4 == 0 && gate_ld % 2 == 0 && ((uintptr_t)gate & 7) == 0) {
+  if (tensor_cores && one_sequence && sh.dk % 8 == 0 && sh.dv % 8 == 0 && out.ld % 2 == 0 && ((uintptr_t)out.out & 7) == 0 && ((uintptr_t)out.out16 & 3) == 0 &&
+      (!out.gate || out.head_gate || (out.gate_ld % 2 == 0 && ((uintptr_t)out.gate & 7) == 0))) {
     int nd = 0, ns = 0;
     MmaKernel kern = mma_kernel(sh.dv, &nd, &ns);
     const bool shared = kv.k == kv.v;
@@ -907,7 +1031,7 @@ cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape&
       cudaError_t e = launch_walk(span_gather_kernel, dim3((keys + 7) / 8, sh.n_kv), dim3(256), 0, s, sh, kv, rows, t0, tokens, L.kr, L.vr, k16, v16);
       if (e != cudaSuccess) return e;
       return launch_walk(kern, dim3((unsigned)(((int64_t)tokens * gq + 63) / 64), sh.n_kv), dim3(128 * ns), smem, s, q, q_ld, sh, (const __half*)k16,
-                         (const __half*)v16, shared, rows, t0, tokens, out, (__nv_bfloat16*)out16, gate, gate_ld);
+                         (const __half*)v16, shared, rows, t0, tokens, out);
     }
   }
   const int groups = (gq + span_heads(sh) - 1) / span_heads(sh), chunk = span_chunk(sh), splits = span_splits(sh), per = span_rows_per_pass(sh);
@@ -923,8 +1047,7 @@ cudaError_t launch_span_attention(const float* q, int64_t q_ld, const SpanShape&
     cudaError_t e = launch_walk(kern, dim3(sh.n_kv * groups, splits, n), dim3(ATT_THREADS), smem, s, q, q_ld, sh, kv, rows, t0 + r, chunk, scratch,
                                 nt && tokens == 1 ? *nt : NewToken{});
     if (e != cudaSuccess) return e;
-    e = launch_walk(span_combine_kernel, dim3(sh.n_head, n, (sh.dv + 127) / 128), dim3(128), 0, s, (const float*)scratch, sh, rows, t0 + r, chunk, splits, out,
-                    (__nv_bfloat16*)out16, gate, gate_ld);
+    e = launch_walk(span_combine_kernel, dim3(sh.n_head, n, (sh.dv + 127) / 128), dim3(128), 0, s, (const float*)scratch, sh, rows, t0 + r, splits, out);
     if (e != cudaSuccess) return e;
   }
   return cudaSuccess;
@@ -937,11 +1060,19 @@ cudaError_t launch_norm_add(float* x, const float* y, int slices, int64_t slice_
   return launch_walk(norm_add_kernel, dim3(tokens), dim3(NORM_ADD_THREADS), 0, s, x, y, slices, slice_stride, w, eps, (__nv_bfloat16*)x16, n);
 }
 
-cudaError_t launch_clamped_glu(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches) {
+cudaError_t launch_add_norm(float* x, const float* y, int slices, int64_t slice_stride, const float* w, float eps, float* h, void* h16, int tokens,
+                            int n, cudaStream_t s, uint64_t* launches) {
+  if (tokens <= 0) return cudaSuccess;
+  if (n % 4 != 0) return cudaErrorInvalidValue;
+  if (launches) ++*launches;
+  return launch_walk(add_norm_kernel, dim3(tokens), dim3(NORM_ADD_THREADS), 0, s, x, y, slices, slice_stride, w, eps, h, (__nv_bfloat16*)h16, n);
+}
+
+cudaError_t launch_gated_unit(const float* gu, const GluShape& sh, float* out, void* out16, int tokens, cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
   const int64_t n = (int64_t)tokens * sh.n / (sh.n % 4 == 0 ? 4 : 1);
-  return launch_walk(clamped_glu_kernel, dim3((unsigned)std::max<int64_t>(1, std::min<int64_t>((n + 255) / 256, 148 * 8))), dim3(256), 0, s, gu, sh, out,
+  return launch_walk(gated_unit_kernel, dim3((unsigned)std::max<int64_t>(1, std::min<int64_t>((n + 255) / 256, 148 * 8))), dim3(256), 0, s, gu, sh, out,
                      (__nv_bfloat16*)out16, tokens);
 }
 

@@ -148,6 +148,8 @@ class Session:
         self._keep = []
         self._adopt(h.value, n_seq, int(cfg["n_vocab"]), int(cfg["n_embd"]), (token_embd, output, layers))
 
+    rewinds = True  # whether a sequence can be truncated to any of its positions
+
     def _adopt(self, handle: int, n_seq: int, n_vocab: int, n_embd: int, model) -> None:
         self._h, self.n_seq, self.n_vocab, self.n_embd = handle, n_seq, n_vocab, n_embd
         self._model = model  # the device reads these matrices for as long as the session lives
@@ -241,7 +243,7 @@ class Session:
 
     def prompt_suffix(self, tokens, seq: int = 0, max_suffix: int = 0):
         """KvCache::prompt_suffix (langtax/src/decode.rs:1155-1195): keeps the longest common prefix of `tokens` and the
-        cached ids, rewinds the cache to it and returns the tokens still to forward, at most max_suffix of them (0: all).
+        cached ids, rewinds the cache to it (to its start where a recurrent state has gone further) and returns the tokens still to forward, at most max_suffix of them (0: all).
         When the whole prompt is cached the last token is forwarded again, so that its logits exist."""
         tokens = [int(v) for v in tokens]
         if not tokens:
@@ -251,6 +253,8 @@ class Session:
         while lcp < len(have) and lcp < len(tokens) and have[lcp] == tokens[lcp]:
             lcp += 1
         keep = len(tokens) - 1 if lcp == len(tokens) else lcp
+        if keep < len(have) and not self.rewinds:
+            keep = 0  # a recurrent state cannot be rewound: the prompt is read again
         self.seq_truncate(seq, keep)
         rest = tokens[keep:]
         return rest[:max_suffix] if max_suffix else rest
@@ -298,8 +302,11 @@ class Session:
             pass
 
 
-MIXER_ATTENTION, MIXER_LATENT = 0, 1
+MIXER_ATTENTION, MIXER_LATENT, MIXER_RETENTION, MIXER_DELTA, MIXER_GATED_LINEAR = range(5)
+NORM_OUTPUT, NORM_INPUT = 0, 1
+UNIT_CLAMPED, UNIT_GELU = 0, 1
 GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
+RECURRENT = (MIXER_RETENTION, MIXER_DELTA, MIXER_GATED_LINEAR)
 
 
 class DecoderSession(Session):
@@ -307,41 +314,56 @@ class DecoderSession(Session):
 
     def __init__(self, executor: "Executor", cfg: dict, token_embd: Matrix, layers, output_norm, pos_embd: Matrix | None = None,
                  output: Matrix | None = None, n_seq: int = 1, kv_blocks: int = 0, block_tokens: int = 16):
-        """cfg: n_embd, n_vocab, n_ctx, norm_eps, embd_scale.  layers: per layer a dict
+        """cfg: n_embd, n_vocab, n_ctx, norm_eps, embd_scale and, where it is not NORM_OUTPUT, norm_place.  layers: per layer a dict
         mixer: kind, n_head, dim, vdim, scale, in, out (Matrix) and, where the mixer has them, n_head_kv, kv_rank, window,
           keep_first, kv_from, gate, up_k, up_v (Matrix), in_bias, q_norm, k_norm, kv_norm (arrays), rel (array
-          [n_bucket, n_head]) and bias_max;
-        mlp: None, or n_ff, limit, alpha, shift, gate_up, down (Matrix);
+          [n_bucket, n_head]) and bias_max, rot_freq (float64 array, an angle per position and pair), sink, width, blocks, taps,
+          decay_rank, gate_rank, unit_eps, gates, decay_up, gate_up (Matrix), conv, conv_bias, gate_bias, decay, step_bias,
+          head_norm (arrays);
+        beside: None, or a second mixer that reads the same input, without in and out; mixer_scale, beside_scale;
+        mlp: None, or n_ff, unit, limit, alpha, shift, gate_up, down (Matrix);
         mixer_norm, mlp_norm: arrays of n_embd."""
         self._exec = executor
         self._h = None
         keep = []
 
-        def host(v):
+        def host(v, dtype=np.float32):
             if v is None:
                 return None
-            keep.append(np.ascontiguousarray(v, np.float32))
+            keep.append(np.ascontiguousarray(v, dtype))
             return keep[-1].ctypes.data
 
         def dev(m):
             return m._h if m is not None else None
+        def mixer(m):
+            rel, freq = m.get("rel"), m.get("rot_freq")
+            return _lib.Mixer(
+                m["kind"], m.get("n_head", 0), m.get("n_head_kv", 0), m.get("dim", 0), m.get("vdim", 0), m.get("kv_rank", 0), m.get("window", 0),
+                m.get("keep_first", 0), m.get("kv_from", -1), m.get("gate", GATE_NONE), float(m["scale"]),
+                0 if rel is None else len(rel), m.get("bias_max", 0), dev(m.get("in")), dev(m.get("up_k")), dev(m.get("up_v")), dev(m.get("out")),
+                host(m.get("in_bias")), host(m.get("q_norm")), host(m.get("k_norm")), host(m.get("kv_norm")), host(rel),
+                0 if freq is None else 2 * len(freq), host(freq, np.float64), host(m.get("sink")),
+                *(m.get(k, 0) for k in ("width", "blocks", "taps", "decay_rank", "gate_rank")), m.get("unit_eps", 0.0),
+                *(dev(m.get(k)) for k in ("gates", "decay_up", "gate_up")),
+                *(host(m.get(k)) for k in ("conv", "conv_bias", "gate_bias", "decay", "step_bias", "head_norm")))
         arr = (_lib.DecoderLayer * len(layers))()
         for i, L in enumerate(layers):
-            m, f = L["mixer"], L.get("mlp")
-            rel = m.get("rel")
-            arr[i].mixer = _lib.Mixer(
-                m["kind"], m["n_head"], m.get("n_head_kv", 0), m["dim"], m["vdim"], m.get("kv_rank", 0), m.get("window", 0),
-                m.get("keep_first", 0), m.get("kv_from", -1), m.get("gate", GATE_NONE), float(m["scale"]),
-                0 if rel is None else len(rel), m.get("bias_max", 0), dev(m["in"]), dev(m.get("up_k")), dev(m.get("up_v")), dev(m["out"]),
-                host(m.get("in_bias")), host(m.get("q_norm")), host(m.get("k_norm")), host(m.get("kv_norm")), host(rel))
+            f, beside = L.get("mlp"), L.get("beside")
+            arr[i].mixer = mixer(L["mixer"])
+            if beside is not None:
+                keep.append(mixer(beside))
+                arr[i].beside = C.pointer(keep[-1])
+                arr[i].mixer_scale, arr[i].beside_scale = L["mixer_scale"], L["beside_scale"]
             if f is not None:
-                arr[i].mlp = _lib.Mlp(f["n_ff"], f["limit"], f["alpha"], f["shift"], dev(f["gate_up"]), dev(f["down"]))
+                arr[i].mlp = _lib.Mlp(f["n_ff"], f.get("unit", UNIT_CLAMPED), f.get("limit", 0.0), f.get("alpha", 0.0), f.get("shift", 0.0),
+                                      dev(f["gate_up"]), dev(f["down"]))
             arr[i].mixer_norm, arr[i].mlp_norm = host(L["mixer_norm"]), host(L.get("mlp_norm"))
-        model = _lib.DecoderModel(len(layers), cfg["n_embd"], cfg["n_vocab"], cfg["n_ctx"], cfg["norm_eps"], cfg["embd_scale"],
+        model = _lib.DecoderModel(len(layers), cfg["n_embd"], cfg["n_vocab"], cfg["n_ctx"], cfg.get("norm_place", NORM_OUTPUT), cfg["norm_eps"], cfg["embd_scale"],
                                   dev(token_embd), dev(pos_embd), dev(output), host(output_norm), arr)
         h = C.c_void_p()
         executor._check(lib().llr_session_create_decoder(executor._h, C.byref(model), n_seq, kv_blocks, block_tokens, C.byref(h)))
         self._adopt(h.value, n_seq, cfg["n_vocab"], cfg["n_embd"], (token_embd, pos_embd, output, layers))
+        self.rewinds = not any(m["kind"] in RECURRENT for L in layers for m in (L["mixer"], L.get("beside")) if m is not None)
 
 
 MOVE_WEIGHTS, DISPATCH_ACTIVATIONS = 0, 1

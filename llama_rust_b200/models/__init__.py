@@ -43,4 +43,4 @@ def load(ex, path, **session_args):
     return _LOADERS[(source, name)](ex, model, **session_args)
 
 
-from . import llama, nagolix  # noqa: E402,F401  (they register themselves)
+from . import llama, mukunex, nagolix  # noqa: E402,F401  (they register themselves)

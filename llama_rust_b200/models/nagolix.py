@@ -8,41 +8,12 @@ from __future__ import annotations
 
 import numpy as np
 
-from ..executor import BF16, DecoderSession, GATE_ELEMENT, GATE_HEAD, MIXER_ATTENTION, MIXER_LATENT
-from ..safetensors import SafetensorsError, SafetensorsFile
+from ..executor import DecoderSession, GATE_ELEMENT, GATE_HEAD, MIXER_ATTENTION, MIXER_LATENT
+from ..safetensors import SafetensorsFile
 from . import register
+from .weights import Weights
 
 GLU_ALPHA, GLU_SHIFT = 1.702, 1.0  # fixed by the design
-
-
-class Weights:
-    """Uploads tensors of one file, stacked by rows where the products of a layer share their input."""
-
-    def __init__(self, ex, file: SafetensorsFile):
-        self.ex, self.file = ex, file
-
-    def stack(self, *parts):
-        """parts: (name, rows, cols); one resident BF16 matrix of all their rows."""
-        for name, rows, cols in parts:
-            self.expect(name, rows, cols)
-            if self.file.dtype(name) != "BF16":
-                raise SafetensorsError(f"{name}: expected BF16, found {self.file.dtype(name)}")
-        raw = [self.file.raw(name) for name, _, _ in parts]
-        return self.ex.upload(BF16, sum(r for _, r, _ in parts), parts[0][2], raw[0] if len(raw) == 1 else np.concatenate(raw))
-
-    def vector(self, name, n):
-        self.expect(name, n)
-        return self.file.f32(name)
-
-    def norm(self, name, n):
-        """A norm weight stored around zero."""
-        return 1.0 + self.vector(name, n)
-
-    def expect(self, name, *shape):
-        if name not in self.file:
-            raise SafetensorsError(f"the file has no tensor {name}")
-        if self.file.shape(name) != shape:
-            raise SafetensorsError(f"{name}: shape {self.file.shape(name)}, the configuration says {shape}")
 
 
 def _latent(w: Weights, p: str, m: dict, width: int) -> dict:
@@ -87,10 +58,10 @@ def load(ex, model, n_ctx=None, **session_args):
         if L["type"] not in MIXERS:
             raise ValueError(f"layer {i}: unknown mixer {L['type']!r}; known: {', '.join(sorted(MIXERS))}")
         mlp = L.get("mlp")
-        layers.append(dict(mixer=MIXERS[L["type"]](w, f"l{i}.mix.", L["mixer"], width), mixer_norm=w.norm(f"l{i}.norm1", width),
+        layers.append(dict(mixer=MIXERS[L["type"]](w, f"l{i}.mix.", L["mixer"], width), mixer_norm=1.0 + w.vector(f"l{i}.norm1", width),
                            mlp=None if mlp is None else _dense(w, f"l{i}.mlp.", mlp, width),
-                           mlp_norm=None if mlp is None else w.norm(f"l{i}.norm2", width)))
+                           mlp_norm=None if mlp is None else 1.0 + w.vector(f"l{i}.norm2", width)))
     return DecoderSession(ex, dict(n_embd=width, n_vocab=vocab, n_ctx=min(n_ctx or positions, positions), norm_eps=cfg["norm"]["eps"],
                                    embd_scale=cfg["embedding"]["scale"]),
-                          w.stack(("embed", vocab, width)), layers, w.norm("final.norm", width), pos_embd=w.stack(("pos", positions, width)),
+                          w.stack(("embed", vocab, width)), layers, 1.0 + w.vector("final.norm", width), pos_embd=w.stack(("pos", positions, width)),
                           **session_args)

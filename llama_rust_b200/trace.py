@@ -51,11 +51,11 @@ def main(argv=None) -> int:
     build.ensure()
     from . import Executor, models
     from .executor import PATH_AUTO, PATH_MMA
-    block = 16
+    block = min(16, a.max_tokens)
     with Executor(0) as ex:
         ex.set_path(PATH_AUTO if a.dtype == "bfloat16" else PATH_MMA)
         # every live request may leave one block partly filled
-        s = models.load(ex, a.model, n_seq=a.max_requests, kv_blocks=-(-a.max_tokens // block) + a.max_requests, block_tokens=block)
+        s = models.load(ex, a.model, n_ctx=a.max_tokens, n_seq=a.max_requests, kv_blocks=-(-a.max_tokens // block) + a.max_requests, block_tokens=block)
         runner = TraceRunner(s, a.out)
         for line in sys.stdin:
             if line.strip():

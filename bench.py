@@ -811,6 +811,45 @@ def layered_session(ex, z, kinds, n_ctx, window, n_seq=1):
                           pos_embd=mat(n_ctx, W), n_seq=n_seq)
 
 
+def mukunex_session(ex, z, kinds, n_ctx, n_seq=1):
+    """A Mukunex-shaped session with random BF16 weights: one layer per entry of `kinds` ("parallel": rotated attention with a
+    sink beside a retention of as many heads as there are key/value heads; "delta": heads of 128 x 128 over the layer's width,
+    half as many query/key heads, ranks 128; "gated": as many blocks as heads)."""
+    from llama_rust_b200 import DTYPES, DecoderSession
+    from llama_rust_b200.executor import (GATE_HEAD, MIXER_ATTENTION, MIXER_DELTA, MIXER_GATED_LINEAR, MIXER_RETENTION, NORM_INPUT, UNIT_GELU)
+    BF16 = DTYPES["BF16"]
+    W, H, G, d = z["width"], z["heads"], z["kv_heads"], z["dim"]
+    seed, rng = [100], np.random.default_rng(1)
+
+    def mat(rows, cols):
+        seed[0] += 1
+        return ex.synth(BF16, rows, cols, seed[0])
+
+    def vec(*shape):
+        return rng.standard_normal(shape).astype(np.float32)
+    ones, layers, freq = np.ones(W, np.float32), [], 5e5 ** (-2.0 * np.arange(d // 2) / d)
+    for kind in kinds:
+        L = dict(mixer_norm=ones, mlp_norm=ones, mlp=dict(n_ff=z["ff"], unit=UNIT_GELU, gate_up=mat(2 * z["ff"], W), down=mat(W, z["ff"])))
+        if kind == "parallel":
+            left, right = (H + 2 * G) * d + H, 4 * G * d
+            m = dict(kind=MIXER_ATTENTION, n_head=H, n_head_kv=G, dim=d, vdim=d, scale=d ** -0.5, gate=GATE_HEAD, rot_freq=freq, sink=vec(H), out=mat(W, (H + G) * d))
+            m["in"] = mat(-(-left // 8) * 8 + right, W)
+            L.update(beside=dict(kind=MIXER_RETENTION, n_head=G, dim=d, vdim=d, scale=d ** -0.5, rot_freq=freq, decay=np.linspace(0.9, 0.9999, G)),
+                     mixer_scale=1.0, beside_scale=1.0)
+        elif kind == "gated":
+            m = dict(kind=MIXER_GATED_LINEAR, width=W, blocks=H, taps=4, scale=8.0, in_bias=vec(2 * W), conv=vec(W, 4), conv_bias=vec(W), gates=mat(2 * W, W // H),
+                     gate_bias=vec(2 * W), decay=vec(W), out=mat(W, W))
+            m["in"] = mat(2 * W, W)
+        else:
+            rows, rank = (H // 2 + H // 2 + H) * d, 128
+            m = dict(kind=MIXER_DELTA, n_head=H, n_head_kv=H // 2, dim=d, vdim=d, scale=d ** -0.5, taps=4, unit_eps=1e-6, decay_rank=rank, gate_rank=rank,
+                     decay_up=mat(H * d, rank), gate_up=mat(H * d, rank), conv=vec(rows, 4), decay=vec(H), step_bias=vec(H * d) - 3, head_norm=vec(d), out=mat(W, H * d))
+            m["in"] = mat(-(-(rows + 2 * rank + H) // 8) * 8, W)
+        layers.append(dict(L, mixer=m))
+    return DecoderSession(ex, dict(n_embd=W, n_vocab=z["vocab"], n_ctx=n_ctx, norm_eps=1e-6, embd_scale=1.0, norm_place=NORM_INPUT), mat(z["vocab"], W), layers, ones,
+                          output=mat(z["vocab"], W), n_seq=n_seq)
+
+
 def llama_session(ex, z, n_layer, n_ctx, n_seq=1):
     """The Llama walk at the same sizes, BF16 weights."""
     from llama_rust_b200 import DTYPES, Session
@@ -829,7 +868,9 @@ def decoder_case(args):
     import torch
     from llama_rust_b200 import Executor, synth
     runs = {"llama": None, "attention": ["attention"] * args.layers, "latent": ["latent"] * args.layers,
-            "mixed": (["latent", "attention", "attention", "shared"] * args.layers)[:args.layers]}
+            "mixed": (["latent", "attention", "attention", "shared"] * args.layers)[:args.layers],
+            "parallel": ["parallel"] * args.layers, "delta": ["delta"] * args.layers, "gated": ["gated"] * args.layers,
+            "recurrent": (["delta", "parallel", "parallel", "gated"] * args.layers)[:args.layers]}
     if args.model:
         runs = {args.model: runs[args.model]}
     out = {"case": "decoder", "layers": args.layers, "prompt": args.prompt, "gen": args.gen, "window": args.window, "data": "synthetic", "dtype": "bf16", "sizes": {}}
@@ -842,7 +883,13 @@ def decoder_case(args):
             ex = Executor(0)
             if args.path is not None:
                 ex.set_path(args.path)
-            s = llama_session(ex, z, args.layers, n_ctx, max(1, args.batch)) if kinds is None else layered_session(ex, z, kinds, n_ctx, args.window, max(1, args.batch))
+            n_seq = max(1, args.batch)
+            if kinds is None:
+                s = llama_session(ex, z, args.layers, n_ctx, n_seq)
+            elif kinds[0] in ("parallel", "delta", "gated"):
+                s = mukunex_session(ex, z, kinds, n_ctx, n_seq)
+            else:
+                s = layered_session(ex, z, kinds, n_ctx, args.window, n_seq)
             prompt = (synth.words(7, 0, args.prompt) % np.uint64(z["vocab"])).astype(np.int32)
             best = [1e9, 1e9]
             for rep in range(args.reps if args.reps != 20 else 4):  # the first is the warm-up
@@ -966,7 +1013,7 @@ def main():
     ap.add_argument("--ctx", type=int, default=0, help="--case session: context length of the session (default: prompt + gen + 8)")
     ap.add_argument("--experts", type=int, default=0, help="--case session: routed experts per layer (0: dense FFN)")
     ap.add_argument("--size", default=None, help="--case decoder: sizes to run, with commas (default: all)")
-    ap.add_argument("--model", default=None, choices=["llama", "attention", "latent", "mixed"], help="--case decoder: one of the models only")
+    ap.add_argument("--model", default=None, choices=["llama", "attention", "latent", "mixed", "parallel", "delta", "gated", "recurrent"], help="--case decoder: one of the models only")
     ap.add_argument("--window", type=int, default=1024, help="--case decoder: window of the layered decoders")
     ap.add_argument("--batch", type=int, default=0, help="--case decoder: also time decode batches over this many sequences")
     args = ap.parse_args()

@@ -1633,7 +1633,7 @@ struct LayeredDecoder {
   size_t block_floats = 0, y_rows = 1, state_floats = 0;
   std::vector<double> freq;  // every distinct rotation, end to end
   float *proj = nullptr, *lat_q = nullptr, *lat_o = nullptr, *att = nullptr, *gu = nullptr, *act = nullptr, *y = nullptr, *scratch = nullptr, *state = nullptr,
-        *prep = nullptr, *low = nullptr;  // low: what the mixers' own products leave
+        *prep = nullptr, *records = nullptr, *low = nullptr;  // low: what the mixers' own products leave
   void *x16 = nullptr, *a16 = nullptr, *b16 = nullptr;
   double* freq_dev = nullptr;
   float2* angles = nullptr;
@@ -1649,7 +1649,7 @@ struct LayeredDecoder {
       if (L.mixer_norm) cudaFree(L.mixer_norm);
       if (L.mlp_norm) cudaFree(L.mlp_norm);
     }
-    float* p[] = {proj, lat_q, lat_o, att, gu, act, y, scratch, state, prep, low};
+    float* p[] = {proj, lat_q, lat_o, att, gu, act, y, scratch, state, prep, records, low};
     for (float* q : p) if (q) cudaFree(q);
     void* v[] = {x16, a16, b16, freq_dev, angles, group_first};
     for (void* q : v) if (q) cudaFree(q);

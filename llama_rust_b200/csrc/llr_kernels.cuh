@@ -448,7 +448,7 @@ struct StateView {
   float* state;
   int64_t stride;
 };
-// Short causal convolution per channel over the rows of a sequence: w [channels][taps], the last tap weighs the row itself.
+// Short causal convolution per channel over the rows of a sequence: w [taps][channels], the last tap weighs the row itself.
 // bias is added to the inputs, out_bias to the results (both may be null); tail: the state's last taps - 1 inputs
 // [taps - 1][channels].
 struct ConvShape {
@@ -485,21 +485,25 @@ struct MatrixScan {
   ConvShape conv;
 };
 bool matrix_scan_supported(int dim, int vdim);
+// Long groups go by blocks of four rows, from records made of their queries, keys and decays (scan_record_floats of them, 16-byte
+// aligned; rows and vectors on 16-byte boundaries).  With `records` the launch takes that form: for retention it makes them, for the
+// delta rule launch_delta_prepare has (q, k, g, beta and kq are not read then).
+bool scan_by_blocks(int dim, int vdim, const RowGroups& groups);
+size_t scan_record_floats(int n_head, int dim, bool delta, int tokens, int n_seq);
 // o_scratch: [tokens][n_head * vdim] floats
-cudaError_t launch_matrix_scan(const MatrixScan& m, const HeadOut& out, const RowGroups& groups, const RowMap& rows, int tokens, float* o_scratch,
-                               cudaStream_t s, uint64_t* launches);
+cudaError_t launch_matrix_scan(const MatrixScan& m, const HeadOut& out, float* records, const RowGroups& groups, const RowMap& rows, int tokens,
+                               float* o_scratch, cudaStream_t s, uint64_t* launches);
 // Inputs of the delta rule from a row of projections q | k | v: convolution, silu, q and k as unit vectors (x / sqrt(sum x^2 +
 // unit_eps)), q times q_scale; g = exp(-rate[h] softplus(a + step_bias)), beta = sigmoid(b).
-// Row t of prep (prep_ld floats): q | k | v | g | beta | k . q.
+// Row t of prep (delta_prep_floats): q | k | v | g | beta | k . q.  With `records`: those, and rows of n_head * vdim values v in prep.
 struct DeltaShape {
   int n_head, n_kv, dim, vdim;
   float q_scale, unit_eps;
   const float *rate, *step_bias;  // [n_head], [n_head * dim]
 };
 int delta_prep_floats(const DeltaShape& d);
-bool delta_supported(const DeltaShape& d);
 cudaError_t launch_delta_prepare(const float* proj, int64_t ld, const float* a, const float* b, const DeltaShape& d, const ConvShape& conv, float* prep,
-                                 const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
+                                 float* records, const RowGroups& groups, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches);
 // u[t] = convolution of the rows at x + t * ld.  u16 (may be null): u as three bfloat16 parts whose sum it is, per block of
 // `block` channels: [channels / block][3][block].
 cudaError_t launch_conv_rows(const float* x, int64_t ld, const ConvShape& conv, float* u, void* u16, int block, const RowMap& rows, int tokens,

@@ -70,7 +70,7 @@ std::string mixer_check(llr_exec* e, const llr_decoder_model* m, size_t li, cons
       return "a part of the delta rule is missing";
     if (!shape(x.decay_up, H * x.dim, x.decay_rank) || !shape(x.gate_up, H * x.vdim, x.gate_rank) || x.decay_up->dtype != LLR_DTYPE_BF16 || x.gate_up->dtype != LLR_DTYPE_BF16)
       return "decay_up / gate_up must be BF16 matrices of n_head * dim / n_head * vdim rows";
-    if (!delta_supported(delta_shape(M))) return "head sizes outside the scan kernels";
+    if (!matrix_scan_supported((int)x.dim, (int)x.vdim)) return "head sizes outside the scan kernels";
     M.channels = (int)(2 * G * x.dim + H * x.vdim);
     M.gate_col = M.channels;  // the low-rank rows: decay, gate; beta behind them
     M.in_rows = M.channels + (int)(x.decay_rank + x.gate_rank + H);
@@ -286,7 +286,8 @@ struct LayeredPass {
     o.gate = proj + M.gate_col;
     o.gate_ld = ld;
     o.silu = true;
-    return launch_matrix_scan(m, o, groups, rows, (int)n, D.low, st, lc);
+    const bool blocks = scan_by_blocks(m.dim, m.vdim, groups) && ld % 4 == 0 && (((uintptr_t)m.q | (uintptr_t)m.k) & 15) == 0;
+    return launch_matrix_scan(m, o, blocks ? D.records : nullptr, groups, rows, (int)n, D.low, st, lc);
   }
 
   // (c) gated delta rule
@@ -314,17 +315,24 @@ struct LayeredPass {
     }
     const DeltaShape d = delta_shape(M);
     const ConvShape conv = convolution(M, nullptr);
-    if ((ce = launch_delta_prepare(proj, ld, a, rank + ra + rg, d, conv, D.prep, rows, N, st, lc)) != cudaSuccess) return ce;
+    const bool blocks = scan_by_blocks(d.dim, d.vdim, groups) && ld % 4 == 0 && ((uintptr_t)proj & 15) == 0;
+    float* records = blocks ? D.records : nullptr;
+    if ((ce = launch_delta_prepare(proj, ld, a, rank + ra + rg, d, conv, D.prep, records, groups, rows, N, st, lc)) != cudaSuccess) return ce;
     MatrixScan m{};
-    m.q = D.prep; m.k = D.prep + nq; m.v = D.prep + 2 * nq; m.g = m.v + nv; m.beta = m.g + ng; m.kq = m.beta + H;
-    m.ld = m.v_ld = delta_prep_floats(d);
+    if (blocks) {
+      m.v = D.prep;
+      m.v_ld = nv;
+    } else {
+      m.q = D.prep; m.k = D.prep + nq; m.v = D.prep + 2 * nq; m.g = m.v + nv; m.beta = m.g + ng; m.kq = m.beta + H;
+      m.ld = m.v_ld = delta_prep_floats(d);
+    }
     m.n_head = H; m.n_kv = (int)mx.n_head_kv; m.dim = (int)mx.dim; m.vdim = (int)mx.vdim;
     m.state = state(M.state_off);
     m.conv_in = proj; m.conv_ld = ld; m.conv = conv;
     HeadOut o = head_out(L, M, out_tc);
     o.gate = gate;
     o.gate_ld = nv;
-    return launch_matrix_scan(m, o, groups, rows, N, o_raw, st, lc);
+    return launch_matrix_scan(m, o, records, groups, rows, N, o_raw, st, lc);
   }
 
   // (d) gated linear recurrence
@@ -450,7 +458,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
   D->norm_input = m->norm_place == LLR_NORM_INPUT;
   D->token_embd = m->token_embd;
   D->pos_embd = m->pos_embd;
-  size_t in_rows = 1, lat = 0, heads = 1, ff = 0, a16 = 8, b16 = 8, scratch = 1, prep = 0, low = 0;
+  size_t in_rows = 1, lat = 0, heads = 1, ff = 0, a16 = 8, b16 = 8, scratch = 1, prep = 0, low = 0, records = 0;
   auto up4 = [](size_t v) { return (v + 3) & ~(size_t)3; };  // vector loads of keys and values
   for (size_t li = 0; li < m->n_layer; ++li) {
     LayeredDecoder::Layer& L = D->layers[li];
@@ -483,6 +491,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
         D->state_floats += up4(channels ? x.width : H * x.dim * x.vdim);
         M.tail_off = (int64_t)D->state_floats;
         if (M.channels > 0) D->state_floats += up4((size_t)(x.taps - 1) * M.channels);
+        if (!channels) records = std::max(records, scan_record_floats((int)H, (int)x.dim, x.kind == LLR_MIXER_DELTA, (int)std::min<size_t>(512, m->n_ctx * n_seq), (int)n_seq));
         if (x.kind == LLR_MIXER_RETENTION) {
           low = std::max(low, H * x.vdim);
         } else if (x.kind == LLR_MIXER_DELTA) {
@@ -536,6 +545,13 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
   cudaError_t ce = cudaSuccess;
   auto alloc = [&](float** p, size_t n) { if (ce == cudaSuccess) ce = cudaMalloc((void**)p, n * sizeof(float)); };
   auto ialloc = [&](int** p, size_t n) { if (ce == cudaSuccess) ce = cudaMalloc((void**)p, n * sizeof(int)); };
+  std::vector<float> by_tap;  // weights of a convolution, [taps][channels]
+  auto taps_first = [&](const float* w, size_t channels, size_t taps) {
+    by_tap.resize(channels * taps);
+    for (size_t c = 0; c < channels; ++c)
+      for (size_t j = 0; j < taps; ++j) by_tap[j * channels + c] = w[c * taps + j];
+    return by_tap.data();
+  };
   auto copy = [&](const float* host, size_t n, float** dev) {
     if (!host || n == 0 || ce != cudaSuccess) return;
     ce = cudaMalloc((void**)dev, n * sizeof(float));
@@ -577,7 +593,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
       } else if (x.kind == LLR_MIXER_DELTA) {
         for (size_t h = 0; h < H; ++h) rate.push_back((float)std::exp((double)x.decay[h]));
         copy(rate.data(), H, &M.decay);
-        copy(x.conv, (size_t)M.channels * x.taps, &M.conv);
+        copy(taps_first(x.conv, M.channels, x.taps), (size_t)M.channels * x.taps, &M.conv);
         copy(x.step_bias, H * x.dim, &M.step_bias);
         copy(x.head_norm, x.vdim, &M.head_norm);
       } else {
@@ -586,7 +602,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
           rate.push_back((float)(x.scale * (z > 0 ? z + std::log1p(std::exp(-z)) : std::log1p(std::exp(z)))));
         }
         copy(rate.data(), x.width, &M.decay);
-        copy(x.conv, (size_t)M.channels * x.taps, &M.conv);
+        copy(taps_first(x.conv, M.channels, x.taps), (size_t)M.channels * x.taps, &M.conv);
         copy(x.conv_bias, x.width, &M.conv_bias);
         copy(x.gate_bias, 2 * (size_t)x.width, &M.gate_bias);
         if (x.in_bias) {
@@ -615,6 +631,7 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
   if (ff) { alloc(&D->gu, B * 2 * ff); alloc(&D->act, B * ff); }
   if (D->state_floats) { alloc(&D->state, n_seq * D->state_floats); alloc(&D->low, B * low + 8); ialloc(&D->group_first, n_seq + 1); }
   if (prep) alloc(&D->prep, B * prep);
+  if (records) alloc(&D->records, records);
   if (!D->freq.empty()) {
     if (ce == cudaSuccess) ce = cudaMalloc((void**)&D->freq_dev, D->freq.size() * sizeof(double));
     if (ce == cudaSuccess) ce = cudaMemcpy(D->freq_dev, D->freq.data(), D->freq.size() * sizeof(double), cudaMemcpyHostToDevice);

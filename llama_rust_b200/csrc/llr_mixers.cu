@@ -129,26 +129,25 @@ __device__ __forceinline__ float rotated(const F& f, int i, int d, const float2*
   const float2 a = cs[c < half ? c : c - half];
   return c < half ? fmaf(v, a.x, -__fmul_rn(f(i + half), a.y)) : fmaf(v, a.x, __fmul_rn(f(i - half), a.y));
 }
-// The same for all n values in place: a pair belongs to one thread.  f(i) reads x[i].
-template <typename F>
-__device__ __forceinline__ void rotate_in_place(const F& f, float* x, int n, int d, const float2* cs, int dims) {
-  const int half = dims / 2, own = d - half;  // a head's pairs, then what passes unchanged
-  for (int j = threadIdx.x; j < n / d * own; j += blockDim.x) {
-    const int c = j % own, i = j / own * d + (c < half ? c : c + half);
-    const float u = f(i);
-    if (c < half) {
-      const float v = f(i + half);
+// The same for `heads` whole heads, a warp per head; put(i, v) takes value i
+template <typename F, typename P>
+__device__ __forceinline__ void rotate_all(const F& f, const P& put, int heads, int d, const float2* cs, int dims) {
+  const int half = dims / 2, lane = threadIdx.x & 31;
+  for (int h = threadIdx.x >> 5; h < heads; h += blockDim.x >> 5) {
+    const int i0 = h * d;
+#pragma unroll 2
+    for (int c = lane; c < half; c += 32) {  // a pair is read and written by one thread
+      const float u = f(i0 + c), v = f(i0 + c + half);
       const float2 a = cs[c];
-      x[i] = fmaf(u, a.x, -__fmul_rn(v, a.y));
-      x[i + half] = fmaf(v, a.x, __fmul_rn(u, a.y));
-    } else {
-      x[i] = u;
+      put(i0 + c, fmaf(u, a.x, -__fmul_rn(v, a.y)));
+      put(i0 + c + half, fmaf(v, a.x, __fmul_rn(u, a.y)));
     }
+    for (int c = dims + lane; c < d; c += 32) put(i0 + c, f(i0 + c));
   }
 }
 __device__ __forceinline__ void rotate_heads(const RotHeads& h, int64_t ld, int t) {
   float* x = h.x + (int64_t)t * ld;
-  rotate_in_place([&](int i) { return x[i]; }, x, h.heads * h.dim, h.dim, h.rot.cs + (int64_t)t * h.rot.ld, h.rot.dims);
+  rotate_all([&](int i) { return x[i]; }, [&](int i, float v) { x[i] = v; }, h.heads, h.dim, h.rot.cs + (int64_t)t * h.rot.ld, h.rot.dims);
 }
 __global__ void __launch_bounds__(256)
 rotate_heads_kernel(RotHeads h, int ld) {
@@ -173,11 +172,15 @@ qkv_store_kernel(float* proj, int ld, const float* __restrict__ bias, const floa
   const float2* cs = rot.dims > 0 ? rot.cs + (int64_t)t * rot.ld : nullptr;
   const auto qf = [&](int i) { return r.q(i); };
   const auto kf = [&](int i) { return r.k(i); };
-  for (int i = threadIdx.x; i < nk; i += PROJ_THREADS)
-    k0[(int64_t)(i / sh.dk) * kv.block_tokens * sh.dk + i % sh.dk] = cs ? rotated(kf, i, sh.dk, cs, rot.dims) : r.k(i);
+  auto k_at = [&](int i) { return k0 + (int64_t)(i / sh.dk) * kv.block_tokens * sh.dk + i % sh.dk; };
+  if (cs) {
+    rotate_all(kf, [&](int i, float v) { *k_at(i) = v; }, sh.n_kv, sh.dk, cs, rot.dims);
+  } else {
+    for (int i = threadIdx.x; i < nk; i += PROJ_THREADS) *k_at(i) = r.k(i);
+  }
   for (int i = threadIdx.x; i < nv; i += PROJ_THREADS) v0[(int64_t)(i / sh.dv) * kv.block_tokens * sh.dv + i % sh.dv] = r.v(i);
   if (cs) {
-    rotate_in_place(qf, p, r.nq, sh.dk, cs, rot.dims);
+    rotate_all(qf, [&](int i, float v) { p[i] = v; }, sh.n_head, sh.dk, cs, rot.dims);
   } else if (bias || q_norm) {
     for (int i0 = threadIdx.x; i0 < r.nq; i0 += 4 * PROJ_THREADS) {  // four values in flight; each is read and written by one thread
       float u[4];

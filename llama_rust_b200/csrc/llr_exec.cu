@@ -16,6 +16,7 @@
 #include <cstdlib>
 #include <atomic>
 #include <cstring>
+#include <functional>
 #include <list>
 #include <memory>
 #include <new>
@@ -1637,6 +1638,8 @@ struct LayeredDecoder {
   void *x16 = nullptr, *a16 = nullptr, *b16 = nullptr;
   double* freq_dev = nullptr;
   float2* angles = nullptr;
+  cudaStream_t side = nullptr;  // of the second of two mixers
+  cudaEvent_t fork = nullptr, join = nullptr;
   int* group_first = nullptr;  // first row of each group of the batch in flight, and their end
   ~LayeredDecoder() {
     for (Layer& L : layers) {
@@ -1653,6 +1656,9 @@ struct LayeredDecoder {
     for (float* q : p) if (q) cudaFree(q);
     void* v[] = {x16, a16, b16, freq_dev, angles, group_first};
     for (void* q : v) if (q) cudaFree(q);
+    if (fork) cudaEventDestroy(fork);
+    if (join) cudaEventDestroy(join);
+    if (side) cudaStreamDestroy(side);
   }
 };
 }  // namespace

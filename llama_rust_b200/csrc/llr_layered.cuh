@@ -163,7 +163,8 @@ struct LayeredPass {
   }
 
   // (a) attention and latent attention: the projection in D.proj becomes result rows in D.att or `h16`
-  cudaError_t attention(const LayeredDecoder::Layer& L, const LayeredDecoder::Mixer& M, bool out_tc, const void** h16) {
+  // `beside` runs once the rows' projections are in place, before the attention itself
+  cudaError_t attention(const LayeredDecoder::Layer& L, const LayeredDecoder::Mixer& M, bool out_tc, const void** h16, const std::function<cudaError_t()>& beside) {
     const llr_mixer& mx = M.mx;
     const int N = (int)n;
     const int64_t ld = L.in_proj->rows;
@@ -197,6 +198,7 @@ struct LayeredPass {
         if (B.mx.kind == LLR_MIXER_RETENTION && B.mx.rot_dims > 0) also = RotHeads{D.proj + B.in_col, 2 * (int)B.mx.n_head, (int)B.mx.dim, rotation(B)};
       if ((ce = launch_qkv_store(proj, (int)ld, M.in_bias, M.q_norm, M.k_norm, sh, rotation(M), also, kv, rows, N, st, lc)) != cudaSuccess) return ce;
     }
+    if ((ce = beside()) != cudaSuccess) return ce;
     // 16-bit result rows where the product that follows takes them: the latent results (lat_o / a16), the heads (att / a16)
     const bool o16 = latent ? up_tc : out_tc;
     SpanOut so{};
@@ -366,6 +368,13 @@ struct LayeredPass {
     return launch_gated_scan(g, groups, rows, N, st, lc);
   }
 
+  cudaError_t mixer(const LayeredDecoder::Layer& L, const LayeredDecoder::Mixer& M, bool out_tc, const void** h16, const std::function<cudaError_t()>& beside) {
+    if (M.mx.kind == LLR_MIXER_RETENTION) return retention(L, M, out_tc);
+    if (M.mx.kind == LLR_MIXER_DELTA) return delta_rule(L, M, out_tc);
+    if (M.mx.kind == LLR_MIXER_GATED_LINEAR) return gated_linear(L, M, out_tc);
+    return attention(L, M, out_tc, h16, beside);
+  }
+
   cudaError_t feed_forward(const LayeredDecoder::Layer& L, const float* h, int* slices) {
     const int N = (int)n, E = (int)s->cfg.n_embd;
     const GluShape glu{(int)L.mlp.n_ff, L.mlp.limit, L.mlp.alpha, L.mlp.shift, (int)L.mlp.unit};
@@ -405,12 +414,21 @@ struct LayeredPass {
       const bool out_tc = tc && L.tc_out;
       if ((ce = before(L.mixer_norm, L.tc_in)) != cudaSuccess || (ce = product(L.in_proj, tc && L.tc_in, h, D.x16, D.proj, nullptr)) != cudaSuccess) return ce;
       const void* h16 = D.a16;
-      for (const LayeredDecoder::Mixer& M : L.mixers) {
-        if (M.mx.kind == LLR_MIXER_RETENTION) ce = retention(L, M, out_tc);
-        else if (M.mx.kind == LLR_MIXER_DELTA) ce = delta_rule(L, M, out_tc);
-        else if (M.mx.kind == LLR_MIXER_GATED_LINEAR) ce = gated_linear(L, M, out_tc);
-        else ce = attention(L, M, out_tc, &h16);
-        if (ce != cudaSuccess) return ce;
+      const std::function<cudaError_t()> nothing = [] { return cudaSuccess; };
+      const bool two = L.mixers.size() == 2 && !L.mixers[0].recurrent && L.mixers[1].recurrent && D.side;
+      if (two) {  // attention and a recurrence: neither fills the machine, so they run next to each other
+        const std::function<cudaError_t()> other = [&] {
+          LayeredPass p{s, n, rows, groups, tc, e, D, D.side, lc};
+          cudaError_t c;
+          if ((c = cudaEventRecord(D.fork, st)) != cudaSuccess || (c = cudaStreamWaitEvent(D.side, D.fork, 0)) != cudaSuccess ||
+              (c = p.mixer(L, L.mixers[1], out_tc, &h16, nothing)) != cudaSuccess)
+            return c;
+          return cudaEventRecord(D.join, D.side);
+        };
+        if ((ce = mixer(L, L.mixers[0], out_tc, &h16, other)) != cudaSuccess || (ce = cudaStreamWaitEvent(st, D.join, 0)) != cudaSuccess) return ce;
+      } else {
+        for (const LayeredDecoder::Mixer& M : L.mixers)
+          if ((ce = mixer(L, M, out_tc, &h16, nothing)) != cudaSuccess) return ce;
       }
       if ((ce = product(L.out_proj, out_tc, D.att, h16, D.y, &slices)) != cudaSuccess || (ce = behind(L.mixer_norm)) != cudaSuccess) return ce;
       if (L.mlp.n_ff == 0) continue;
@@ -631,6 +649,12 @@ int layered_create(llr_exec* e, const llr_decoder_model* m, size_t n_seq, size_t
   if (ff) { alloc(&D->gu, B * 2 * ff); alloc(&D->act, B * ff); }
   if (D->state_floats) { alloc(&D->state, n_seq * D->state_floats); alloc(&D->low, B * low + 8); ialloc(&D->group_first, n_seq + 1); }
   if (prep) alloc(&D->prep, B * prep);
+  for (const auto& L : D->layers)
+    if (L.mixers.size() == 2 && !D->side && ce == cudaSuccess) {
+      ce = cudaStreamCreateWithFlags(&D->side, cudaStreamNonBlocking);
+      if (ce == cudaSuccess) ce = cudaEventCreateWithFlags(&D->fork, cudaEventDisableTiming);
+      if (ce == cudaSuccess) ce = cudaEventCreateWithFlags(&D->join, cudaEventDisableTiming);
+    }
   if (records) alloc(&D->records, records);
   if (!D->freq.empty()) {
     if (ce == cudaSuccess) ce = cudaMalloc((void**)&D->freq_dev, D->freq.size() * sizeof(double));

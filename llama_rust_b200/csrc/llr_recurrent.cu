@@ -53,18 +53,25 @@ __device__ __forceinline__ float conv_at(const float* x, int64_t ld, const ConvS
   }
   return cv.out_bias ? __fadd_rn(acc, cv.out_bias[c]) : acc;
 }
-// channels c .. c + 3, all on 16-byte boundaries, no biases: the same sums
+// channels c .. c + 3, all on 16-byte boundaries: the same sums
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(__fadd_rn(a.x, b.x), __fadd_rn(a.y, b.y), __fadd_rn(a.z, b.z), __fadd_rn(a.w, b.w)); }
 __device__ __forceinline__ float4 conv4_at(const float* x, int64_t ld, const ConvShape& cv, const float* tail, int t, int near, int pos, int c) {
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  const float4 b = cv.bias ? *(const float4*)(cv.bias + c) : acc;
 #pragma unroll 4
   for (int j = cv.taps - 1; j >= 0; --j) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (j <= near) v = *(const float4*)(x + (int64_t)(t - j) * ld + c);
-    else if (j <= pos) v = *(const float4*)(tail + (int64_t)(cv.taps - 1 - (j - near)) * cv.channels + c);
+    if (j <= near) {
+      v = *(const float4*)(x + (int64_t)(t - j) * ld + c);
+      if (cv.bias) v = add4(v, b);
+    }
+    else if (j <= pos) {
+      v = *(const float4*)(tail + (int64_t)(cv.taps - 1 - (j - near)) * cv.channels + c);
+    }
     const float4 w = *(const float4*)(cv.w + (int64_t)(cv.taps - 1 - j) * cv.channels + c);
     acc = make_float4(fmaf(w.x, v.x, acc.x), fmaf(w.y, v.y, acc.y), fmaf(w.z, v.z, acc.z), fmaf(w.w, v.w, acc.w));
   }
-  return acc;
+  return cv.out_bias ? add4(acc, *(const float4*)(cv.out_bias + c)) : acc;
 }
 __device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 __device__ __forceinline__ float4 silu4(float4 z) { return make_float4(silu(z.x), silu(z.y), silu(z.z), silu(z.w)); }
@@ -75,36 +82,64 @@ __device__ __forceinline__ void conv_tail_update(const float* x, int64_t ld, con
   const int keep = cv.taps - 1, n = g.t1 - g.t0;
   for (int c = at; c < cv.channels; c += all) {
     const float b = cv.bias ? cv.bias[c] : 0.f;
-    for (int k = 0; k < keep; ++k) {  // ascending: what moves down is read before it is written
-      const int back = keep - k;      // rows before the next one
-      float v;
-      if (back <= n) v = __fadd_rn(x[(int64_t)(g.t1 - back) * ld + c], b);
-      else v = g.fresh ? 0.f : tail[(int64_t)(k + n) * cv.channels + c];
-      tail[(int64_t)k * cv.channels + c] = v;
+    for (int k0 = 0; k0 < keep; k0 += 4) {  // ascending: what moves down is read before it is written
+      float v[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int k = k0 + j, back = keep - k;  // rows before the next one
+        v[j] = 0.f;
+        if (k < keep) {
+          if (back <= n) v[j] = __fadd_rn(x[(int64_t)(g.t1 - back) * ld + c], b);
+          else if (!g.fresh) v[j] = tail[(int64_t)(k + n) * cv.channels + c];
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (k0 + j < keep) tail[(int64_t)(k0 + j) * cv.channels + c] = v[j];
     }
   }
 }
 
-// one block per row and CONV_COLS channels
-constexpr int CONV_COLS = 256;
-__global__ void __launch_bounds__(256)
-conv_rows_kernel(const float* __restrict__ x, int64_t ld, ConvShape cv, float* __restrict__ u, __nv_bfloat16* __restrict__ u16, int block, RowMap rows) {
+// v as a sum of three bfloat16 values: 24 bits of mantissa
+__device__ __forceinline__ void in_parts(float v, __nv_bfloat16 (&p)[3]) {
+  p[0] = __float2bfloat16_rn(v);
+  v = __fsub_rn(v, __bfloat162float(p[0]));
+  p[1] = __float2bfloat16_rn(v);
+  p[2] = __float2bfloat16_rn(__fsub_rn(v, __bfloat162float(p[1])));
+}
+// grid (row, CONV_COLS channels); vec: four channels per thread, everything on boundaries of four
+constexpr int CONV_THREADS = 128;
+__global__ void __launch_bounds__(CONV_THREADS)
+conv_rows_kernel(const float* __restrict__ x, int64_t ld, ConvShape cv, float* __restrict__ u, __nv_bfloat16* __restrict__ u16, int block, RowMap rows, bool vec) {
   pdl_enter();
-  const int t = blockIdx.x, near = rows_before(rows, t, cv.taps - 1), pos = row_position(rows, t);
+  const int t = blockIdx.x, near = rows_before(rows, t, cv.taps - 1), pos = row_position(rows, t), at = blockIdx.y * CONV_THREADS + threadIdx.x;
   const float* tail = cv.tail.state + row_sequence(rows, t) * cv.tail.stride;
-  const int c1 = min(cv.channels, (int)(blockIdx.y + 1) * CONV_COLS);
-  for (int c = blockIdx.y * CONV_COLS + threadIdx.x; c < c1; c += 256) {
-    const float v = conv_at(x, ld, cv, tail, t, near, pos, c);
-    u[(int64_t)t * cv.channels + c] = v;
-    if (u16) {  // v as a sum of three bfloat16 values: 24 bits of mantissa
+  if (vec) {
+    const int c = 4 * at;
+    if (c >= cv.channels) return;
+    const float4 v = conv4_at(x, ld, cv, tail, t, near, pos, c);
+    *(float4*)(u + (int64_t)t * cv.channels + c) = v;
+    if (u16) {
+      __nv_bfloat16 p[4][3];
+      in_parts(v.x, p[0]); in_parts(v.y, p[1]); in_parts(v.z, p[2]); in_parts(v.w, p[3]);
       __nv_bfloat16* o = u16 + (int64_t)t * 3 * cv.channels + (int64_t)(c / block) * 3 * block + c % block;
-      const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-      const float r1 = __fsub_rn(v, __bfloat162float(hi));
-      const __nv_bfloat16 mid = __float2bfloat16_rn(r1);
-      o[0] = hi;
-      o[block] = mid;
-      o[2 * block] = __float2bfloat16_rn(__fsub_rn(r1, __bfloat162float(mid)));
+#pragma unroll
+      for (int k = 0; k < 3; ++k) {
+        const __nv_bfloat162 lo = __halves2bfloat162(p[0][k], p[1][k]), hi = __halves2bfloat162(p[2][k], p[3][k]);
+        *(uint2*)(o + k * block) = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+      }
     }
+    return;
+  }
+  if (at >= cv.channels) return;
+  const float v = conv_at(x, ld, cv, tail, t, near, pos, at);
+  u[(int64_t)t * cv.channels + at] = v;
+  if (u16) {
+    __nv_bfloat16 p[3];
+    in_parts(v, p);
+    __nv_bfloat16* o = u16 + (int64_t)t * 3 * cv.channels + (int64_t)(at / block) * 3 * block + at % block;
+#pragma unroll
+    for (int k = 0; k < 3; ++k) o[k * block] = p[k];
   }
 }
 
@@ -118,51 +153,45 @@ __global__ void triple_columns_kernel(const uint16_t* __restrict__ w, int64_t n,
 // ---- inputs of the delta rule -------------------------------------------------------------------------------------------
 __device__ __forceinline__ float fade(float rate, float a, float bias) { return expf(-__fmul_rn(rate, softplus(__fadd_rn(a, bias)))); }
 
-// a warp per row and key/value head: the head's query and key, and values, decays and step of the heads that share them
-__global__ void __launch_bounds__(128)
+// grid (row, key/value head), a thread per value where they fit a block: the head's query and key, and values and decays of the
+// heads that share them
+__global__ void __launch_bounds__(1024)
 delta_prepare_kernel(const float* __restrict__ proj, int64_t ld, const float* __restrict__ a, const float* __restrict__ b, DeltaShape d, ConvShape cv,
-                     float* __restrict__ prep, int64_t prep_ld, RowMap rows, int tokens) {
+                     float* __restrict__ prep, int64_t prep_ld, RowMap rows) {
   pdl_enter();
-  const int lane = threadIdx.x & 31, w = blockIdx.x * 4 + (threadIdx.x >> 5), t = w / d.n_kv, kvh = w % d.n_kv;
-  if (t >= tokens) return;
-  const int near = rows_before(rows, t, cv.taps - 1), pos = row_position(rows, t), share = d.n_head / d.n_kv;
+  extern __shared__ float qk[];  // the head's q | k behind convolution and silu
+  __shared__ float red[3][32];
+  const int t = blockIdx.x, kvh = blockIdx.y, near = rows_before(rows, t, cv.taps - 1), pos = row_position(rows, t), share = d.n_head / d.n_kv;
   const float* tail = cv.tail.state + row_sequence(rows, t) * cv.tail.stride;
   const int nq = d.n_kv * d.dim, nv = d.n_head * d.vdim, ng = d.n_head * d.dim;
+  const int end_v = 2 * d.dim + share * d.vdim, end = end_v + share * d.dim;
   float* o = prep + (int64_t)t * prep_ld;
-  const float* at = a + (int64_t)t * ng;
-  auto active = [&](int c) { return silu(conv_at(proj, ld, cv, tail, t, near, pos, c)); };
-  float *oq = o + kvh * d.dim, *ok = oq + nq;
   float sq = 0.f, sk = 0.f;
-#pragma unroll 2
-  for (int i = lane; i < d.dim; i += 32) {
-    const float q = active(kvh * d.dim + i), k = active(nq + kvh * d.dim + i);
-    oq[i] = q;  // read again below by the lane that wrote it
-    ok[i] = k;
-    sq = fmaf(q, q, sq);
-    sk = fmaf(k, k, sk);
+  for (int i = threadIdx.x; i < end; i += blockDim.x) {
+    if (i < end_v) {
+      const int c = i < d.dim ? kvh * d.dim + i : i < 2 * d.dim ? nq + kvh * d.dim + i - d.dim : 2 * nq + kvh * share * d.vdim + i - 2 * d.dim;
+      const float v = silu(conv_at(proj, ld, cv, tail, t, near, pos, c));
+      if (i < 2 * d.dim) qk[i] = v;
+      else o[c] = v;
+      if (i < d.dim) sq = fmaf(v, v, sq);
+      else if (i < 2 * d.dim) sk = fmaf(v, v, sk);
+    } else {
+      const int c = kvh * share * d.dim + i - end_v;
+      o[2 * nq + nv + c] = fade(d.rate[c / d.dim], a[(int64_t)t * ng + c], d.step_bias[c]);
+    }
   }
-#pragma unroll 2
-  for (int i = lane; i < share * d.vdim; i += 32) {
-    const int c = 2 * nq + kvh * share * d.vdim + i;
-    o[c] = active(c);
-  }
-  for (int h = kvh * share; h < (kvh + 1) * share; ++h) {
-    const float rate = d.rate[h];
-#pragma unroll 2
-    for (int c = h * d.dim + lane; c < (h + 1) * d.dim; c += 32) o[2 * nq + nv + c] = fade(rate, at[c], d.step_bias[c]);
-    if (lane == 0) o[2 * nq + nv + ng + h] = sigmoid(b[(int64_t)t * ld + h]);
-  }
-  sq = sqrtf(__fadd_rn(warp_sum(sq), d.unit_eps));
-  sk = sqrtf(__fadd_rn(warp_sum(sk), d.unit_eps));
+  for (int j = threadIdx.x; j < share; j += blockDim.x) o[2 * nq + nv + ng + kvh * share + j] = sigmoid(b[(int64_t)t * ld + kvh * share + j]);
+  sq = sqrtf(__fadd_rn(block_sum(sq, red[0]), d.unit_eps));
+  sk = sqrtf(__fadd_rn(block_sum(sk, red[1]), d.unit_eps));
   float kq = 0.f;
-  for (int i = lane; i < d.dim; i += 32) {
-    const float qv = __fmul_rn(__fdiv_rn(oq[i], sq), d.q_scale), kv = __fdiv_rn(ok[i], sk);
-    oq[i] = qv;
-    ok[i] = kv;
+  for (int i = threadIdx.x; i < d.dim; i += blockDim.x) {  // qk is complete: the sums have synchronized
+    const float qv = __fmul_rn(__fdiv_rn(qk[i], sq), d.q_scale), kv = __fdiv_rn(qk[d.dim + i], sk);
+    o[kvh * d.dim + i] = qv;
+    o[nq + kvh * d.dim + i] = kv;
     kq = fmaf(kv, qv, kq);
   }
-  kq = warp_sum(kq);
-  if (lane == 0) o[2 * nq + nv + ng + d.n_head + kvh] = kq;
+  kq = block_sum(kq, red[2]);
+  if (threadIdx.x == 0) o[2 * nq + nv + ng + d.n_head + kvh] = kq;
 }
 
 // ---- four rows at a time ------------------------------------------------------------------------------------------------
@@ -195,68 +224,62 @@ __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(
 __device__ __forceinline__ float4 mul4(float4 a, float b) { return make_float4(a.x * b, a.y * b, a.z * b, a.w * b); }
 __device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
 
-// a warp per block and head, a lane per four key channels
-__global__ void __launch_bounds__(128)
+// grid (block of rows, head), a warp per row, a lane per four key channels
+__global__ void __launch_bounds__(32 * BLOCK_ROWS)
 delta_blocks_kernel(const float* __restrict__ proj, int64_t ld, const float* __restrict__ a, const float* __restrict__ b, DeltaShape d, ConvShape cv,
-                    int dp, float* __restrict__ rec, float* __restrict__ v_out, RowGroups groups, RowMap rows, int tokens, int slots) {
+                    int dp, float* __restrict__ rec, float* __restrict__ v_out, RowGroups groups, RowMap rows, int tokens) {
   pdl_enter();
-  const int lane = threadIdx.x & 31, w = blockIdx.x * 4 + (threadIdx.x >> 5), slot = w / d.n_head, h = w % d.n_head, kvh = h / (d.n_head / d.n_kv);
-  if (slot >= slots) return;
+  __shared__ float4 sq[BLOCK_ROWS][32], sk[BLOCK_ROWS][32], sg[BLOCK_ROWS][32];
+  const int lane = threadIdx.x & 31, i = threadIdx.x >> 5, slot = blockIdx.x, h = blockIdx.y, kvh = h / (d.n_head / d.n_kv);
   const BlockAt at = block_at(groups, tokens, slot);
   if (at.n <= 0) return;
-  const int nq = d.n_kv * d.dim, nv = d.n_head * d.vdim, ng = d.n_head * d.dim, c = 4 * lane;
-  const float* tail = cv.tail.state + row_sequence(rows, at.t0) * cv.tail.stride;
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  const bool on = c < d.dim;
-  const float rate = d.rate[h];
-  float4 q[4], k[4], g[4];
-#pragma unroll
-  for (int r = 0; r < 4; ++r) {
-    q[r] = k[r] = zero;
-    g[r] = make_float4(1.f, 1.f, 1.f, 1.f);
-    if (r < at.n) {
-      const int t = at.t0 + r, near = rows_before(rows, t, cv.taps - 1), pos = row_position(rows, t);
-      if (on) {
-        q[r] = silu4(conv4_at(proj, ld, cv, tail, t, near, pos, kvh * d.dim + c));
-        k[r] = silu4(conv4_at(proj, ld, cv, tail, t, near, pos, nq + kvh * d.dim + c));
-        const float4 s = *(const float4*)(a + (int64_t)t * ng + h * d.dim + c), bias = *(const float4*)(d.step_bias + h * d.dim + c);
-        g[r] = make_float4(fade(rate, s.x, bias.x), fade(rate, s.y, bias.y), fade(rate, s.z, bias.z), fade(rate, s.w, bias.w));
-      }
-      for (int i = c; i < d.vdim; i += 128)
-        *(float4*)(v_out + (int64_t)t * nv + h * d.vdim + i) = silu4(conv4_at(proj, ld, cv, tail, t, near, pos, 2 * nq + h * d.vdim + i));
-      q[r] = mul4(q[r], __fdiv_rn(d.q_scale, sqrtf(__fadd_rn(warp_sum(dot4(q[r], q[r])), d.unit_eps))));
-      k[r] = mul4(k[r], __fdiv_rn(1.0f, sqrtf(__fadd_rn(warp_sum(dot4(k[r], k[r])), d.unit_eps))));
-    }
-  }
+  const int nq = d.n_kv * d.dim, nv = d.n_head * d.vdim, ng = d.n_head * d.dim, c = 4 * lane, t = at.t0 + i;
+  float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q, g = make_float4(1.f, 1.f, 1.f, 1.f);
   float* o = rec + ((int64_t)slot * d.n_head + h) * rec_floats(dp, true);
   float* sc = o + rec_vectors(true) * dp;
-  auto put = [&](int i, float4 v) { if (c < dp) *(float4*)(o + i * dp + c) = v; };
-  float4 p = g[0];
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    if (i > 0) p = mul4(p, g[i]);
-    put(i, mul4(p, k[i]));
-    put(4 + i, mul4(p, q[i]));
-  }
-  put(12, p);
-#pragma unroll
-  for (int j = 0; j < 4; ++j) {  // k_j faded up to row i, read by rows i >= j
-    float4 f = k[j];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      float cij = 0.f, sij = 0.f;
-      if (i >= j) {
-        if (i > j) {
-          f = mul4(f, g[i]);
-          cij = warp_sum(dot4(f, k[i]));
-        }
-        sij = warp_sum(dot4(f, q[i]));
-      }
-      if (lane == 0) { sc[4 * i + j] = sij; sc[16 + 4 * i + j] = cij; }
+  if (i < at.n) {
+    const int near = rows_before(rows, t, cv.taps - 1), pos = row_position(rows, t);
+    const float* tail = cv.tail.state + row_sequence(rows, t) * cv.tail.stride;
+    if (c < d.dim) {
+      const float rate = d.rate[h];
+      const float4 s = *(const float4*)(a + (int64_t)t * ng + h * d.dim + c), bias = *(const float4*)(d.step_bias + h * d.dim + c);
+      q = silu4(conv4_at(proj, ld, cv, tail, t, near, pos, kvh * d.dim + c));
+      k = silu4(conv4_at(proj, ld, cv, tail, t, near, pos, nq + kvh * d.dim + c));
+      g = make_float4(fade(rate, s.x, bias.x), fade(rate, s.y, bias.y), fade(rate, s.z, bias.z), fade(rate, s.w, bias.w));
     }
-    put(8 + j, f);
+    for (int j = c; j < d.vdim; j += 128)
+      *(float4*)(v_out + (int64_t)t * nv + h * d.vdim + j) = silu4(conv4_at(proj, ld, cv, tail, t, near, pos, 2 * nq + h * d.vdim + j));
+    q = mul4(q, __fdiv_rn(d.q_scale, sqrtf(__fadd_rn(warp_sum(dot4(q, q)), d.unit_eps))));
+    k = mul4(k, __fdiv_rn(1.0f, sqrtf(__fadd_rn(warp_sum(dot4(k, k)), d.unit_eps))));
   }
-  if (lane < 4) sc[32 + lane] = lane < at.n ? sigmoid(b[(int64_t)(at.t0 + lane) * ld + h]) : 0.f;
+  sq[i][lane] = q;
+  sk[i][lane] = k;
+  sg[i][lane] = g;
+  if (lane == 0) sc[32 + i] = i < at.n ? sigmoid(b[(int64_t)t * ld + h]) : 0.f;
+  __syncthreads();
+  // row i against the rows up to it: k_j faded from j to i, the last j first
+  float4 f = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+  for (int j = BLOCK_ROWS - 1; j >= 0; --j) {
+    float sij = 0.f, cij = 0.f;
+    if (j <= i) {
+      const float4 kj = mul4(f, sk[j][lane]);
+      sij = warp_sum(dot4(kj, q));
+      if (j < i) cij = warp_sum(dot4(kj, k));
+      f = mul4(f, sg[j][lane]);
+    }
+    if (lane == 0) { sc[4 * i + j] = sij; sc[16 + 4 * i + j] = cij; }
+  }
+  // f: all decays up to row i; the decays behind it
+  float4 after = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+  for (int j = 1; j < BLOCK_ROWS; ++j)
+    if (j > i) after = mul4(after, sg[j][lane]);
+  auto put = [&](int at, float4 v) { if (c < dp) *(float4*)(o + at * dp + c) = v; };
+  put(i, mul4(f, k));
+  put(BLOCK_ROWS + i, mul4(f, q));
+  put(2 * BLOCK_ROWS + i, mul4(after, k));
+  if (i == BLOCK_ROWS - 1) put(3 * BLOCK_ROWS, f);
 }
 
 // the same for retention, from rotated queries and keys
@@ -372,7 +395,6 @@ matrix_scan_kernel(MatrixScan m, HeadOut ho, RowGroups groups, RowMap rows, int 
   const Group g = group_of(groups, rows, tokens, blockIdx.z);
   const int tid = threadIdx.x, nt = blockDim.x, l = tid % LPC, col = tid / LPC * C, head = blockIdx.y, kvh = head / (m.n_head / m.n_kv);
   const int c0 = blockIdx.x * cols, live = min(cols, m.vdim - c0), stage = L::stage(cols), v_ld = (cols + 3) & ~3;
-  if (DELTA) conv_tail_update(m.conv_in, m.conv_ld, m.conv, g, (blockIdx.y * gridDim.x + blockIdx.x) * nt + tid, (int)(gridDim.x * gridDim.y) * nt);
   if (m.dim < DP) {  // values behind dim stay zero
     for (int i = tid; i < SCAN_STAGES * stage; i += nt) sm[i] = 0.f;
     __syncthreads();
@@ -455,6 +477,7 @@ matrix_scan_kernel(MatrixScan m, HeadOut ho, RowGroups groups, RowMap rows, int 
       S[c][j] = make_pair(v.x, v.y);
       S[c][j + 1] = make_pair(v.z, v.w);
     }
+  if (DELTA) conv_tail_update(m.conv_in, m.conv_ld, m.conv, g, (blockIdx.y * gridDim.x + blockIdx.x) * nt + tid, (int)(gridDim.x * gridDim.y) * nt);
   const pair decay = DELTA ? 0 : both(m.decay[head]);
   float* o_row = o_raw + ((int64_t)g.t0 * m.n_head + head) * m.vdim + c0 + col;
   const int64_t o_ld = (int64_t)m.n_head * m.vdim;
@@ -591,7 +614,6 @@ block_scan_kernel(MatrixScan m, RowGroups groups, RowMap rows, int tokens, int c
   const int my_c = l / REP / 4, my_i = l / REP % 4;  // the product this lane ends up with
   float* xd = sm + BLOCK_STAGES * stage + grp * V;
   float* xu = xd + nt / LPC * V;
-  if (DELTA) conv_tail_update(m.conv_in, m.conv_ld, m.conv, g, (blockIdx.y * gridDim.x + blockIdx.x) * nt + tid, (int)(gridDim.x * gridDim.y) * nt);
   const int n = g.t1 - g.t0, steps = (n + BLOCK_ROWS - 1) / BLOCK_ROWS;
   const float* src = rec + ((int64_t)first_block(groups, blockIdx.z) * m.n_head + head) * L::REC;
   const float* v_row = m.v + (int64_t)g.t0 * m.v_ld + (int64_t)head * m.vdim + c0;
@@ -633,6 +655,7 @@ block_scan_kernel(MatrixScan m, RowGroups groups, RowMap rows, int tokens, int c
       S[c][j] = v.x;
       S[c][j + 1] = v.y;
     }
+  if (DELTA) conv_tail_update(m.conv_in, m.conv_ld, m.conv, g, (blockIdx.y * gridDim.x + blockIdx.x) * nt + tid, (int)(gridDim.x * gridDim.y) * nt);
   // sums over the lanes of V values; the lane's own one is returned
   auto spread = [&](float (&val)[V]) {
     int w = V;
@@ -858,19 +881,23 @@ cudaError_t launch_delta_prepare(const float* proj, int64_t ld, const float* a, 
   if (records) {
     if (!scan_by_blocks(d.dim, d.vdim, groups) || ld % 4 != 0 || (((uintptr_t)proj | (uintptr_t)a) & 15) != 0) return cudaErrorInvalidValue;
     const int slots = block_slots(tokens, groups.n);
-    return launch_walk(delta_blocks_kernel, dim3((unsigned)(((int64_t)slots * d.n_head + 3) / 4)), dim3(128), 0, s, proj, ld, a, b, d, conv,
-                       padded_dim(d.dim), records, prep, groups, rows, tokens, slots);
+    return launch_walk(delta_blocks_kernel, dim3(slots, d.n_head), dim3(32 * BLOCK_ROWS), 0, s, proj, ld, a, b, d, conv, padded_dim(d.dim), records, prep, groups,
+                       rows, tokens);
   }
-  return launch_walk(delta_prepare_kernel, dim3((unsigned)(((int64_t)tokens * d.n_kv + 3) / 4)), dim3(128), 0, s, proj, ld, a, b, d, conv, prep,
-                     (int64_t)delta_prep_floats(d), rows, tokens);
+  const int share = d.n_head / d.n_kv, values = 2 * d.dim + share * (d.dim + d.vdim);
+  return launch_walk(delta_prepare_kernel, dim3(tokens, d.n_kv), dim3(std::min(1024, (values + 31) / 32 * 32)), (size_t)2 * d.dim * sizeof(float), s, proj, ld, a,
+                     b, d, conv, prep, (int64_t)delta_prep_floats(d), rows);
 }
 
 cudaError_t launch_conv_rows(const float* x, int64_t ld, const ConvShape& conv, float* u, void* u16, int block, const RowMap& rows, int tokens,
                              cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
-  return launch_walk(conv_rows_kernel, dim3(tokens, (conv.channels + CONV_COLS - 1) / CONV_COLS), dim3(256), 0, s, x, ld, conv, u, (__nv_bfloat16*)u16, block,
-                     rows);
+  const bool vec = ((conv.channels | block | (int)ld) & 3) == 0 &&
+                   (((uintptr_t)x | (uintptr_t)u | (uintptr_t)conv.bias | (uintptr_t)conv.tail.state) & 15) == 0 && conv.tail.stride % 4 == 0;
+  const int per = CONV_THREADS * (vec ? 4 : 1);
+  return launch_walk(conv_rows_kernel, dim3(tokens, (conv.channels + per - 1) / per), dim3(CONV_THREADS), 0, s, x, ld, conv, u, (__nv_bfloat16*)u16, block, rows,
+                     vec);
 }
 
 cudaError_t launch_triple_columns(const void* w, int64_t rows, int cols, void* out, cudaStream_t s, uint64_t* launches) {
@@ -903,9 +930,10 @@ static cudaError_t launch_block_scan(const MatrixScan& m, const HeadOut& out, fl
     if (e != cudaSuccess) return e;
   }
   if (launches) *launches += 2;
-  e = launch_walk(c.kern, dim3((m.vdim + cols - 1) / cols, m.n_head, groups.n), dim3(threads), smem, s, m, groups, rows, tokens, cols, (const float*)records,
-                  o_scratch);
-  if (e != cudaSuccess) return e;
+  // Not placed while its predecessor runs, unlike the walk's other kernels: one block per SM for long is the whole plan, and blocks
+  // that start early crowd onto the SMs that happen to be free.
+  c.kern<<<dim3((m.vdim + cols - 1) / cols, m.n_head, groups.n), threads, smem, s>>>(m, groups, rows, tokens, cols, records, o_scratch);
+  if ((e = cudaGetLastError()) != cudaSuccess) return e;
   return launch_walk(head_out_kernel, dim3((unsigned)(((int64_t)tokens * m.n_head + 7) / 8)), dim3(256), 0, s, (const float*)o_scratch, m.n_head, m.vdim, out,
                      tokens);
 }
@@ -942,7 +970,10 @@ cudaError_t launch_matrix_scan(const MatrixScan& m, const HeadOut& out, float* r
 cudaError_t launch_gated_scan(const GatedScan& g, const RowGroups& groups, const RowMap& rows, int tokens, cudaStream_t s, uint64_t* launches) {
   if (tokens <= 0) return cudaSuccess;
   if (launches) ++*launches;
-  return launch_walk(gated_scan_kernel, dim3((g.width + GS_COLS - 1) / GS_COLS, groups.n), dim3(GS_COLS * GS_LANES), 0, s, g, groups, rows, tokens);
+  const dim3 grid((g.width + GS_COLS - 1) / GS_COLS, groups.n);
+  if (groups.longest <= SCAN_SHORT) return launch_walk(gated_scan_kernel, grid, dim3(GS_COLS * GS_LANES), 0, s, g, groups, rows, tokens);
+  gated_scan_kernel<<<grid, GS_COLS * GS_LANES, 0, s>>>(g, groups, rows, tokens);  // not placed early, as above
+  return cudaGetLastError();
 }
 
 }  // namespace llr

@@ -802,15 +802,16 @@ gated_scan_kernel(GatedScan p, RowGroups groups, RowMap rows, int tokens) {
       const int r = first + j * GS_LANES;
       if (r >= n) break;
       const float log_a = -__fmul_rn(rate, sigmoid(__fadd_rn(gr[j], rb)));
-      const float in = sqrtf(-expm1f(2.0f * log_a));  // sqrt(1 - a^2) without the cancellation near a = 1
-      ab[r][lane] = make_float2(expf(log_a), __fmul_rn(__fmul_rn(in, sigmoid(__fadd_rn(gi[j], ib))), u[j]));
+      // a - 1 instead of a: a state that hardly fades would feel every rounding of a factor next to 1, at each of its steps
+      const float less = expm1f(log_a), in = sqrtf(-__fmul_rn(less, 2.0f + less));  // 1 - a^2 = -(a - 1) (a + 1)
+      ab[r][lane] = make_float2(less, __fmul_rn(__fmul_rn(in, sigmoid(__fadd_rn(gi[j], ib))), u[j]));
     }
     __syncthreads();
     if (runs) {
 #pragma unroll 8
       for (int r = 0; r < n; ++r) {
         const float2 v = ab[r][lane];
-        S = fmaf(v.x, S, v.y);
+        S = __fadd_rn(S, fmaf(v.x, S, v.y));
         ab[r][lane].x = S;
       }
     }

@@ -175,6 +175,22 @@ def test_long_decoding(ex, stock, path):
     s.free()
 
 
+def test_states_that_hardly_fade(ex, tmp_path):
+    """Decays next to 1 over a thousand positions: the recurrences' rounding must not add up."""
+    cfg = mm.config(64, 60, [mm.rglru(96, 3, 4), mm.parallel((2, 1, 16, 16, R8, 0.25), (2, 16, 16, R8, [0.9999, 1.0])), mm.delta(2, 1, 16, 16, 4)], 0)
+    w = mm.weights(cfg, 31)
+    w["l0.mix.lam"] = mm.rounded(w["l0.mix.lam"] - 5.0)
+    w["l2.mix.dt_bias"] = mm.rounded(w["l2.mix.dt_bias"] - 4.0)
+    toks = mm.tokens(1100, cfg, 14)
+    want = plain.forward(cfg, w, toks)
+    s = _open(ex, mm.write(tmp_path / "m", cfg, w), mm.F32, n_ctx=1100)
+    for sizes in ([1100], [1000, 1]):
+        s.reset()
+        e = mm.error(_feed(s, 0, toks, sizes), want)
+        assert e.max() <= 2e-5, e.max()
+    s.free()
+
+
 @pytest.mark.parametrize("path", PATHS)
 def test_prompt_longer_than_a_batch(ex, stock, path):
     cfg, _, folder, logits = stock("tiles")
@@ -315,6 +331,30 @@ def test_batches_of_unequal_requests(ex, stock, name, path):
             at[i] += take[i]
     for i, r in enumerate(reqs):
         _close(np.concatenate(got[i]), logits(r), path, f"request {i}")
+    s.free()
+
+
+def test_f32_rows_do_not_depend_on_their_batch(ex, stock):
+    cfg, _, folder, _ = stock("mix")
+    a, b = mm.tokens(40, cfg, 50), mm.tokens(23, cfg, 51)
+    s = _open(ex, folder, mm.F32, n_seq=2)
+    alone = [_feed(s, q, t, [10 ** 6]) for q, t in ((0, a), (1, b))]
+    s.reset()
+    both = s.forward([(1, b), (0, a)], [list(range(23)), list(range(40))])
+    assert mm.error(both[:23], alone[1].astype(np.float64)).max() < 2e-6 and mm.error(both[23:], alone[0].astype(np.float64)).max() < 2e-6
+    s.free()
+
+
+def test_a_long_prompt_beside_many_sequences(ex, stock):
+    """More groups than the scans take by blocks: 70 sequences, one of them with a long portion."""
+    cfg, _, folder, logits = stock("mix")
+    reqs = [mm.tokens(40 if q == 33 else 3, cfg, 300 + q) for q in range(70)]
+    s = _open(ex, folder, mm.F32, n_ctx=64, n_seq=70)
+    for lo, hi in ((0, 2), (2, 40)):
+        live = [q for q in range(70) if len(reqs[q]) > lo]
+        out = s.forward([(q, reqs[q][lo:hi]) for q in live], [[len(reqs[q][lo:hi]) - 1] for q in live])
+        for k, q in enumerate(live):
+            _close(out[k:k + 1], logits(reqs[q][:hi])[-1:], mm.F32, f"sequence {q}")
     s.free()
 
 

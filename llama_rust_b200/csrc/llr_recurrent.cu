@@ -333,19 +333,54 @@ __device__ __forceinline__ void async16(float* dst, const float* src) {
 __device__ __forceinline__ void async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// a head's result behind its norm and gate; a warp per head and row.  o: vdim values in shared or global memory
+// a head's result behind its norm and gate; a warp per head and row
 __device__ __forceinline__ void head_out(const float* o, int vdim, const HeadOut& ho, int t, int h, int lane) {
+  const float* gate = ho.gate + (int64_t)t * ho.gate_ld + (int64_t)h * vdim;
+  const int64_t at = (int64_t)t * ho.ld + (int64_t)h * vdim;
+  auto inverse = [&](float ss) { return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(warp_sum(ss), (float)vdim), ho.eps))); };
+  auto value = [&](float v, float inv, int i, float g) {
+    v = __fmul_rn(v, inv);
+    if (ho.weight) v = __fmul_rn(v, ho.weight[i]);
+    return __fmul_rn(__fmul_rn(v, ho.silu ? __fmul_rn(g, sigmoid(g)) : sigmoid(g)), ho.scale);
+  };
+  __nv_bfloat16* out16 = (__nv_bfloat16*)ho.out16;
+  const bool vec = (vdim & 3) == 0 && vdim <= 256 && (((uintptr_t)o | (uintptr_t)gate) & 15) == 0 && (!ho.out || ((uintptr_t)(ho.out + at) & 15) == 0) &&
+                   (!out16 || ((uintptr_t)(out16 + at) & 7) == 0);
+  if (vec) {  // the whole head at once
+    float4 v[2], g[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = 4 * (lane + 32 * j);
+      if (i < vdim) {
+        v[j] = *(const float4*)(o + i);
+        g[j] = *(const float4*)(gate + i);
+        ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, ss))));
+      }
+    }
+    const float inv = inverse(ss);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = 4 * (lane + 32 * j);
+      if (i < vdim) {
+        const float4 r = make_float4(value(v[j].x, inv, i, g[j].x), value(v[j].y, inv, i + 1, g[j].y), value(v[j].z, inv, i + 2, g[j].z),
+                                     value(v[j].w, inv, i + 3, g[j].w));
+        if (ho.out) *(float4*)(ho.out + at + i) = r;
+        if (out16) {
+          const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+          *(uint2*)(out16 + at + i) = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+        }
+      }
+    }
+    return;
+  }
   float ss = 0.f;
   for (int i = lane; i < vdim; i += 32) ss = fmaf(o[i], o[i], ss);
-  const float rms = sqrtf(__fadd_rn(__fdiv_rn(warp_sum(ss), (float)vdim), ho.eps));
+  const float inv = inverse(ss);
   for (int i = lane; i < vdim; i += 32) {
-    float v = __fdiv_rn(o[i], rms);
-    if (ho.weight) v = __fmul_rn(v, ho.weight[i]);
-    const float g = ho.gate[(int64_t)t * ho.gate_ld + (int64_t)h * vdim + i];
-    v = __fmul_rn(__fmul_rn(v, ho.silu ? __fmul_rn(g, sigmoid(g)) : sigmoid(g)), ho.scale);
-    const int64_t at = (int64_t)t * ho.ld + (int64_t)h * vdim + i;
-    if (ho.out) ho.out[at] = v;
-    if (ho.out16) ((__nv_bfloat16*)ho.out16)[at] = __float2bfloat16_rn(v);
+    const float v = value(o[i], inv, i, gate[i]);
+    if (ho.out) ho.out[at + i] = v;
+    if (out16) out16[at + i] = __float2bfloat16_rn(v);
   }
 }
 __global__ void __launch_bounds__(256)
